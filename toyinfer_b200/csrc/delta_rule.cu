@@ -1,4 +1,4 @@
-// The gated delta rule with one decay per key channel, and the per-head gated norm after it.
+// The gated delta rule with one decay per key channel or one per head, and the per-head gated norm after it.
 //
 // Per head, with a state S [dim, vdim] in float32 that a sequence carries from token to token
 // (zero when the sequence starts), a unit query q and key k [dim], a value v [vdim], a write
@@ -7,7 +7,8 @@
 // in this order, so that the read-out sees the token's own write.  Query and key arrive unnormalised
 // (after their short convolution and silu) and are made unit vectors here, x / sqrt(sum x^2 + 1e-6),
 // the query also times dim^-1/2.  The decay comes as the logit l of a low-rank projection:
-// g = exp(-rate_h * softplus(l + dt)), rate_h = exp(A_h) made once.  beta = sigmoid of its logit.
+// g = exp(-rate_h * softplus(l + dt)), rate_h = exp(A_h) made once; with one decay per head (head_decay) l and dt are one
+// number per head and the whole state takes the same g.  beta = sigmoid of its logit.
 // Value head h reads query/key head h / (heads / qk_heads).  Everything of the recurrence is 32-bit.
 //
 // delta_rule_prep makes unit q and k, decays and betas of all the step's tokens at once.
@@ -37,9 +38,10 @@ constexpr int DR_LPC = 16, DR_COLS = 8, DR_THREADS = DR_LPC * DR_COLS;      // s
 // What the recurrence needs of every token, made for all tokens at once: one warp per (token, unit); units 0 .. G - 1 are
 // the query/key heads (unit vectors qn, kn [M, G, dim], the query times dim^-1/2), units G .. G + H - 1 the value heads
 // (decays g [M, H, dim] and beta [M, H]).  All float32.
-template <typename T>
+// L: type of the decay logits.  HEAD: one decay per head (gg [M, H]).
+template <typename T, typename L, bool HEAD>
 __global__ void delta_rule_prep_kernel(const T* __restrict__ q, const T* __restrict__ k, long long q_stride, long long k_stride,
-                                       const float* __restrict__ decay_logit, const float* __restrict__ dt_bias,
+                                       const L* __restrict__ decay_logit, long long decay_stride, const float* __restrict__ dt_bias,
                                        const float* __restrict__ rate, const T* __restrict__ beta_logit, long long beta_stride,
                                        float* __restrict__ qn, float* __restrict__ kn, float* __restrict__ gg, float* __restrict__ beta,
                                        long long rows, int n_heads, int qk_heads, int dim) {
@@ -67,9 +69,13 @@ __global__ void delta_rule_prep_kernel(const T* __restrict__ q, const T* __restr
     } else {
         const int h = unit - qk_heads;
         const float rt = rate[h];
-        const float* l = decay_logit + ((size_t)m * n_heads + h) * dim;
-        float* go = gg + ((size_t)m * n_heads + h) * dim;
-        for (int i = lane; i < dim; i += 32) go[i] = expf(-rt * softplus_f(l[i] + dt_bias[(size_t)h * dim + i]));
+        if constexpr (HEAD) {
+            if (lane == 0) gg[(size_t)m * n_heads + h] = expf(-rt * softplus_f(to_f32(decay_logit[(size_t)m * decay_stride + h]) + dt_bias[h]));
+        } else {
+            const L* l = decay_logit + (size_t)m * decay_stride + (size_t)h * dim;
+            float* go = gg + ((size_t)m * n_heads + h) * dim;
+            for (int i = lane; i < dim; i += 32) go[i] = expf(-rt * softplus_f(to_f32(l[i]) + dt_bias[(size_t)h * dim + i]));
+        }
         if (lane == 0) beta[(size_t)m * n_heads + h] = 1.0f / (1.0f + expf(-to_f32(beta_logit[(size_t)m * beta_stride + h])));
     }
 }
@@ -91,7 +97,8 @@ __device__ __forceinline__ FloatRun<N> lds_run(const float* p) {
     return out;
 }
 
-template <typename T, int MAXD>
+// (HEAD: one decay per head; only q and k are staged as rows then, and the decays ride beside the betas.)
+template <typename T, int MAXD, bool HEAD>
 __global__ void __launch_bounds__(DR_THREADS)
 delta_rule_scan_kernel(const float* __restrict__ qn, const float* __restrict__ kn, const float* __restrict__ gg,
                        const float* __restrict__ beta, const T* __restrict__ v, long long v_stride,
@@ -100,16 +107,17 @@ delta_rule_scan_kernel(const float* __restrict__ qn, const float* __restrict__ k
                        int n_heads, int qk_heads, int dim, int vdim, int groups) {
     ti_pdl_trigger();
     constexpr int NV = MAXD / DR_LPC >= 4 ? 4 : MAXD / DR_LPC, J = MAXD / (DR_LPC * NV), ROW = MAXD;
-    constexpr int PIECES = 3 * DR_TOK * ROW / 4;                         // 16-byte pieces of a run's q, k, g
+    constexpr int PIECES = (HEAD ? 2 : 3) * DR_TOK * ROW / 4;            // 16-byte pieces of a run's q, k, g
     constexpr int PER = (PIECES + DR_THREADS - 1) / DR_THREADS;
-    extern __shared__ __align__(16) float sm[];                  // q, k, g: [DR_TOK][ROW] each; v: [DR_TOK][DR_COLS]; beta: [DR_TOK]
+    extern __shared__ __align__(16) float sm[];                  // q, k, g: [DR_TOK][ROW] each; v: [DR_TOK][DR_COLS]; beta, decay: [DR_TOK]
     ti_pdl_sync();
     qn = ti_dependent(qn); kn = ti_dependent(kn); gg = ti_dependent(gg); beta = ti_dependent(beta); v = ti_dependent(v);
     float* qs = sm;
     float* ks = qs + DR_TOK * ROW;
     float* gs = ks + DR_TOK * ROW;
-    float* vs = gs + DR_TOK * ROW;
+    float* vs = HEAD ? gs : gs + DR_TOK * ROW;
     float* bs = vs + DR_TOK * DR_COLS;
+    float* ds = bs + DR_TOK;
     const int h = blockIdx.x / groups, g = blockIdx.x - h * groups;
     const int b = blockIdx.y;
     const int tok0 = cu_new[b], n = cu_new[b + 1] - tok0;
@@ -135,7 +143,7 @@ delta_rule_scan_kernel(const float* __restrict__ qn, const float* __restrict__ k
             S[jj][e] = i < dim ? sm[i * DR_COLS + cl] : 0.f;
         }
     float4 rr[PER];
-    float rv = 0.f, rb = 0.f;
+    float rv = 0.f, rb = 0.f, rd = 0.f;
     auto fetch = [&](int t0) {
         const int nt = min(DR_TOK, n - t0);
 #pragma unroll
@@ -164,7 +172,10 @@ delta_rule_scan_kernel(const float* __restrict__ qn, const float* __restrict__ k
             const int tt = threadIdx.x / DR_COLS, c = g * DR_COLS + (threadIdx.x - tt * DR_COLS);
             rv = (tt < nt && c < vdim) ? to_f32(v[(size_t)(tok0 + t0 + tt) * v_stride + (size_t)h * vdim + c]) : 0.f;
         }
-        if (threadIdx.x < DR_TOK) rb = threadIdx.x < nt ? beta[(size_t)(tok0 + t0 + threadIdx.x) * n_heads + h] : 0.f;
+        if (threadIdx.x < DR_TOK) {
+            rb = threadIdx.x < nt ? beta[(size_t)(tok0 + t0 + threadIdx.x) * n_heads + h] : 0.f;
+            if constexpr (HEAD) rd = threadIdx.x < nt ? gg[(size_t)(tok0 + t0 + threadIdx.x) * n_heads + h] : 0.f;
+        }
     };
     fetch(0);
     for (int t0 = 0; t0 < n; t0 += DR_TOK) {
@@ -174,7 +185,10 @@ delta_rule_scan_kernel(const float* __restrict__ qn, const float* __restrict__ k
         for (int p = 0; p < PER; p++)
             if (threadIdx.x + DR_THREADS * p < PIECES) reinterpret_cast<float4*>(sm)[threadIdx.x + DR_THREADS * p] = rr[p];
         if (threadIdx.x < DR_TOK * DR_COLS) vs[threadIdx.x] = rv;
-        if (threadIdx.x < DR_TOK) bs[threadIdx.x] = rb;
+        if (threadIdx.x < DR_TOK) {
+            bs[threadIdx.x] = rb;
+            if constexpr (HEAD) ds[threadIdx.x] = rd;
+        }
         __syncthreads();
         if (t0 + DR_TOK < n) fetch(t0 + DR_TOK);          // on its way while this run is worked off
         // Token by token.  A warp issues in order, so the loop is arranged by hand: the next token's q, k, g are read
@@ -184,28 +198,31 @@ delta_rule_scan_kernel(const float* __restrict__ qn, const float* __restrict__ k
 #pragma unroll
             for (int jj = 0; jj < J; jj++) x[jj] = lds_run<NV>(base + tt * ROW + DR_LPC * NV * jj + NV * r);
         };
-        auto decay_and_dot = [&](const FloatRun<NV> (&gv)[J], const FloatRun<NV> (&kv)[J]) {
+        auto decay_and_dot = [&](const FloatRun<NV> (&gv)[HEAD ? 1 : J], float gh, const FloatRun<NV> (&kv)[J]) {
             float d0 = 0.f, d1 = 0.f;
 #pragma unroll
             for (int jj = 0; jj < J; jj++)
 #pragma unroll
                 for (int e = 0; e < NV; e++) {
-                    S[jj][e] *= gv[jj].x[e];
+                    if constexpr (HEAD) S[jj][e] *= gh; else S[jj][e] *= gv[jj].x[e];
                     if (e & 1) d1 = fmaf(S[jj][e], kv[jj].x[e], d1); else d0 = fmaf(S[jj][e], kv[jj].x[e], d0);
                 }
             return d0 + d1;
         };
-        FloatRun<NV> kc[J], qc[J], gc[J];
-        rows_of(ks, 0, kc); rows_of(qs, 0, qc); rows_of(gs, 0, gc);
-        float dot = decay_and_dot(gc, kc);
+        FloatRun<NV> kc[J], qc[J], gc[HEAD ? 1 : J];
+        rows_of(ks, 0, kc); rows_of(qs, 0, qc);
+        float gh = 0.f;
+        if constexpr (HEAD) gh = ds[0]; else rows_of(gs, 0, gc);
+        float dot = decay_and_dot(gc, gh, kc);
         float bv = bs[0], vv = vs[cl];
 #pragma unroll
         for (int sh = 1; sh < DR_LPC; sh <<= 1) dot += __shfl_xor_sync(0xffffffffu, dot, sh);
         for (int tt = 0; tt < nt; tt++) {
             const bool more = tt + 1 < nt;
             const int nx = more ? tt + 1 : tt;
-            FloatRun<NV> kx[J], qx[J], gx[J];
-            rows_of(ks, nx, kx); rows_of(qs, nx, qx); rows_of(gs, nx, gx);
+            FloatRun<NV> kx[J], qx[J], gx[HEAD ? 1 : J];
+            rows_of(ks, nx, kx); rows_of(qs, nx, qx);
+            if constexpr (HEAD) gh = ds[nx]; else rows_of(gs, nx, gx);
             const float bn = bs[nx], vn = vs[nx * DR_COLS + cl];
             const float e = bv * (vv - dot);
             float a0 = 0.f, a1 = 0.f;
@@ -218,7 +235,7 @@ delta_rule_scan_kernel(const float* __restrict__ qn, const float* __restrict__ k
                 }
             float acc = a0 + a1;
             float nd = 0.f;
-            if (more) nd = decay_and_dot(gx, kx);            // (the same for all lanes)
+            if (more) nd = decay_and_dot(gx, gh, kx);            // (the same for all lanes)
 #pragma unroll
             for (int sh = 1; sh < DR_LPC; sh <<= 1) {
                 acc += __shfl_xor_sync(0xffffffffu, acc, sh);
@@ -274,44 +291,68 @@ template <typename F>
 int dispatch_dim(int dim, F&& f) {
     if (dim <= 32) return f(std::integral_constant<int, 32>());
     if (dim <= 64) return f(std::integral_constant<int, 64>());
-    return f(std::integral_constant<int, 128>());
+    if (dim <= 128) return f(std::integral_constant<int, 128>());
+    return f(std::integral_constant<int, 256>());
 }
 
 }  // namespace
 
-// q, k: [M, qk_heads, dim] and v: [M, heads, vdim] of the engine's type (row strides given, heads dense); decay_logit:
-// float32 [M, heads * dim]; dt_bias: float32 [heads * dim]; rate: float32 [heads]; beta_logit: [M, heads] (row stride
-// given); o: float32 [M, heads * vdim]; state: float32, slot s at state + s * slot_stride holds [heads, dim, vdim];
-// scratch: float32, M * (2 * qk_heads * dim + heads * dim + heads) values.
-extern "C" int ti_delta_rule_scan(const void* q, const void* k, const void* v, long long q_stride, long long k_stride,
-                                  long long v_stride, const float* decay_logit, const float* dt_bias, const float* rate,
-                                  const void* beta_logit, long long beta_stride, float* o, float* state, long long slot_stride,
-                                  float* scratch, const int* cu_new, const int* seq_slot, int n_seq, int M, int n_heads,
-                                  int qk_heads, int dim, int vdim, int dtype, cudaStream_t stream) {
-    if (n_seq == 0 || M == 0) return 0;
-    TI_REQUIRE(n_seq > 0 && n_seq <= 65535 && M > 0 && n_heads > 0 && qk_heads > 0 && n_heads % qk_heads == 0 && dim > 0 && vdim > 0 && scratch,
-               "delta_rule_scan: bad sizes");
-    TI_REQUIRE(dim <= 128, "delta_rule: heads of %d query/key elements are not supported (up to 128)", dim);
+namespace {
+
+template <typename T, typename L, bool HEAD>
+int delta_rule_run(const void* q, const void* k, const void* v, long long q_stride, long long k_stride, long long v_stride,
+                   const void* decay_logit, long long decay_stride, const float* dt_bias, const float* rate, const void* beta_logit,
+                   long long beta_stride, float* o, float* state, long long slot_stride, float* scratch, const int* cu_new,
+                   const int* seq_slot, int n_seq, int M, int n_heads, int qk_heads, int dim, int vdim, cudaStream_t stream) {
     const int groups = (vdim + DR_COLS - 1) / DR_COLS;
     float* qn = scratch;
     float* kn = qn + (size_t)M * qk_heads * dim;
     float* gg = kn + (size_t)M * qk_heads * dim;
-    float* beta = gg + (size_t)M * n_heads * dim;
+    float* beta = gg + (size_t)M * n_heads * (HEAD ? 1 : dim);
     const long long rows = (long long)M * (qk_heads + n_heads);
+    TI_CUDA(ti_launch(delta_rule_prep_kernel<T, L, HEAD>, dim3((unsigned)((rows + 3) / 4)), dim3(128), 0, stream, (const T*)q, (const T*)k,
+                      q_stride, k_stride, (const L*)decay_logit, decay_stride, dt_bias, rate, (const T*)beta_logit, beta_stride, qn, kn, gg,
+                      beta, rows, n_heads, qk_heads, dim));
+    TI_CHECK_LAUNCH("delta_rule_prep");
+    return dispatch_dim(dim, [&](auto md) -> int {
+        constexpr int MAXD = decltype(md)::value;
+        constexpr size_t smem = (size_t)((HEAD ? 2 : 3) * DR_TOK * MAXD + 2 * DR_TOK + DR_TOK * DR_COLS) * sizeof(float);
+        static_assert(smem >= (size_t)MAXD * DR_COLS * sizeof(float), "a block's columns of the state pass through the same memory");
+        if constexpr (smem > 48 * 1024)
+            TI_CUDA(cudaFuncSetAttribute(delta_rule_scan_kernel<T, MAXD, HEAD>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+        TI_CUDA(ti_launch(delta_rule_scan_kernel<T, MAXD, HEAD>, dim3(n_heads * groups, n_seq), dim3(DR_THREADS), smem, stream,
+                          (const float*)qn, (const float*)kn, (const float*)gg, (const float*)beta, (const T*)v, v_stride, o, state,
+                          slot_stride, cu_new, seq_slot, n_heads, qk_heads, dim, vdim, groups));
+        TI_CHECK_LAUNCH("delta_rule_scan");
+        return 0;
+    });
+}
+
+}  // namespace
+
+// q, k: [M, qk_heads, dim] and v: [M, heads, vdim] of the engine's type (row strides given, heads dense); head_decay 0:
+// decay_logit float32 [M, heads * dim], dt_bias float32 [heads * dim]; head_decay 1: decay_logit [M, heads] of the engine's
+// type, dt_bias float32 [heads] (row stride decay_stride in both); rate: float32 [heads]; beta_logit: [M, heads] (row stride
+// given); o: float32 [M, heads * vdim]; state: float32, slot s at state + s * slot_stride holds [heads, dim, vdim];
+// scratch: float32, M * (2 * qk_heads * dim + heads * (head_decay ? 1 : dim) + heads) values, 16-byte aligned.
+extern "C" int ti_delta_rule_scan(const void* q, const void* k, const void* v, long long q_stride, long long k_stride,
+                                  long long v_stride, const void* decay_logit, long long decay_stride, int head_decay,
+                                  const float* dt_bias, const float* rate, const void* beta_logit, long long beta_stride, float* o,
+                                  float* state, long long slot_stride, float* scratch, const int* cu_new, const int* seq_slot, int n_seq,
+                                  int M, int n_heads, int qk_heads, int dim, int vdim, int dtype, cudaStream_t stream) {
+    if (n_seq == 0 || M == 0) return 0;
+    TI_REQUIRE(n_seq > 0 && n_seq <= 65535 && M > 0 && n_heads > 0 && qk_heads > 0 && n_heads % qk_heads == 0 && dim > 0 && vdim > 0 && scratch,
+               "delta_rule_scan: bad sizes");
+    TI_REQUIRE(dim <= 256, "delta_rule: heads of %d query/key elements are not supported (up to 256)", dim);
     return ti_dispatch_dtype(dtype, [&](auto t) -> int {
         using T = decltype(t);
-        TI_CUDA(ti_launch(delta_rule_prep_kernel<T>, dim3((unsigned)((rows + 3) / 4)), dim3(128), 0, stream, (const T*)q, (const T*)k, q_stride,
-                          k_stride, decay_logit, dt_bias, rate, (const T*)beta_logit, beta_stride, qn, kn, gg, beta, rows, n_heads, qk_heads, dim));
-        TI_CHECK_LAUNCH("delta_rule_prep");
-        return dispatch_dim(dim, [&](auto md) -> int {
-            constexpr int MAXD = decltype(md)::value;
-            constexpr size_t smem = (size_t)(3 * DR_TOK * MAXD + DR_TOK + DR_TOK * DR_COLS) * sizeof(float);
-            TI_CUDA(ti_launch(delta_rule_scan_kernel<T, MAXD>, dim3(n_heads * groups, n_seq), dim3(DR_THREADS), smem, stream,
-                              (const float*)qn, (const float*)kn, (const float*)gg, (const float*)beta, (const T*)v, v_stride, o, state,
-                              slot_stride, cu_new, seq_slot, n_heads, qk_heads, dim, vdim, groups));
-            TI_CHECK_LAUNCH("delta_rule_scan");
-            return 0;
-        });
+        if (head_decay)
+            return delta_rule_run<T, T, true>(q, k, v, q_stride, k_stride, v_stride, decay_logit, decay_stride, dt_bias, rate, beta_logit,
+                                              beta_stride, o, state, slot_stride, scratch, cu_new, seq_slot, n_seq, M, n_heads, qk_heads, dim,
+                                              vdim, stream);
+        return delta_rule_run<T, float, false>(q, k, v, q_stride, k_stride, v_stride, decay_logit, decay_stride, dt_bias, rate, beta_logit,
+                                               beta_stride, o, state, slot_stride, scratch, cu_new, seq_slot, n_seq, M, n_heads, qk_heads,
+                                               dim, vdim, stream);
     });
 }
 

@@ -7,7 +7,8 @@
 // place i, off[e] .. off[e + 1] the places of expert e.  One block.
 //
 // moe_route_softmax: the same output for a router with softmax scores s = softmax(z) over all experts.  Experts are
-// CHOSEN by s + correction (a float32 value per expert, or none), only among the experts of the `keep` best of
+// CHOSEN by s + correction (a float32 value per expert; without one by the logits themselves, which keep the order also
+// where scores underflow; a bias per expert may be added to the logits first), only among the experts of the `keep` best of
 // `n_groups` equal runs of neighbouring experts (a run's score is its largest choice score; n_groups <= 1: all
 // experts), ties to the lower index; a pair's WEIGHT is its s divided by the sum of the token's chosen s (+ 1e-20),
 // times `scale`.  Scores that are not allowed do not count as 0: choice scores may be negative.
@@ -90,7 +91,8 @@ __device__ __forceinline__ void group_pairs(int* cnt, int* offs, int* cur, int n
 
 constexpr int MAX_GROUPS = 64;
 
-__global__ void moe_route_softmax_kernel(const float* __restrict__ z, long long ldz, const float* __restrict__ correction,
+__global__ void moe_route_softmax_kernel(const float* __restrict__ z, long long ldz, const float* __restrict__ logit_bias,
+                                         const float* __restrict__ correction,
                                          int n_experts, int top, int n_groups, int keep, float scale, int M,
                                          int* __restrict__ perm, int* __restrict__ off, int* __restrict__ pair_expert,
                                          float* __restrict__ pair_w) {
@@ -105,13 +107,14 @@ __global__ void moe_route_softmax_kernel(const float* __restrict__ z, long long 
     const int per = n_groups > 1 ? n_experts / n_groups : n_experts;
     for (int m = threadIdx.x; m < M; m += blockDim.x) {
         const float* zr = z + (size_t)m * ldz;
+        auto logit = [&](int e) { return zr[e] + (logit_bias ? logit_bias[e] : 0.f); };
         float zmax = -INFINITY;
-        for (int e = 0; e < n_experts; e++) zmax = fmaxf(zmax, zr[e]);
+        for (int e = 0; e < n_experts; e++) zmax = fmaxf(zmax, logit(e));
         float sum = 0.f;
-        for (int e = 0; e < n_experts; e++) sum += expf(zr[e] - zmax);
+        for (int e = 0; e < n_experts; e++) sum += expf(logit(e) - zmax);
         const float inv = 1.0f / sum;
-        auto score = [&](int e) { return expf(zr[e] - zmax) * inv; };
-        auto choice = [&](int e) { return score(e) + (correction ? correction[e] : 0.f); };
+        auto score = [&](int e) { return expf(logit(e) - zmax) * inv; };
+        auto choice = [&](int e) { return correction ? score(e) + correction[e] : logit(e); };
         unsigned long long open = ~0ull;                 // bit g: experts of run g may be chosen
         if (n_groups > 1 && keep < n_groups) {
             open = 0ull;
@@ -196,9 +199,9 @@ extern "C" int ti_moe_route_topk(const float* z, long long ldz, int n_experts, i
     return 0;
 }
 
-// z: float32 [M, >= n_experts] with row stride ldz; correction: float32 [n_experts] or null; n_groups <= 1: no runs; perm: int32
+// z: float32 [M, >= n_experts] with row stride ldz; logit_bias, correction: float32 [n_experts] or null; n_groups <= 1: no runs; perm: int32
 // [M * top]; off: int32 [n_experts + 1]; pair_expert: int32 scratch [M * top]; pair_w: float32 [M * top].
-extern "C" int ti_moe_route_softmax(const float* z, long long ldz, const float* correction, int n_experts, int top, int n_groups,
+extern "C" int ti_moe_route_softmax(const float* z, long long ldz, const float* logit_bias, const float* correction, int n_experts, int top, int n_groups,
                                     int keep, float scale, int M, int* perm, int* off, int* pair_expert, float* pair_w,
                                     cudaStream_t stream) {
     if (M == 0) return 0;
@@ -211,8 +214,8 @@ extern "C" int ti_moe_route_softmax(const float* z, long long ldz, const float* 
                    top, MAX_GROUPS);
     const size_t smem = (size_t)(3 * n_experts + 1) * sizeof(int);
     TI_REQUIRE(smem <= 48 * 1024, "moe_route_softmax: %d experts are too many", n_experts);
-    TI_CUDA(ti_launch_class<1>(moe_route_softmax_kernel, dim3(1), dim3(RT_THREADS), smem, stream, z, ldz, correction, n_experts, top,
-                               n_groups, keep, scale, M, perm, off, pair_expert, pair_w));
+    TI_CUDA(ti_launch_class<1>(moe_route_softmax_kernel, dim3(1), dim3(RT_THREADS), smem, stream, z, ldz, logit_bias, correction, n_experts,
+                               top, n_groups, keep, scale, M, perm, off, pair_expert, pair_w));
     TI_CHECK_LAUNCH("moe_route_softmax");
     return 0;
 }

@@ -12,14 +12,24 @@ from .wide import _fn
 P, I, L, F = c_void_p, c_int, c_longlong, c_float
 
 
+POINTWISE_ACTS = {"relu2": 0, "gelu": 1}
+
+
+def pointwise_act(x: torch.Tensor, act: str) -> torch.Tensor:
+    """An ungated activation, elementwise in 32-bit with one rounding: "relu2" max(x, 0)^2, "gelu" x (1 + erf(x / sqrt(2))) / 2."""
+    _need_cuda(x, what="pointwise_act")
+    if act not in POINTWISE_ACTS:
+        raise KernelError(f"pointwise_act: unknown activation {act!r}; known: {sorted(POINTWISE_ACTS)}")
+    if not x.is_contiguous():
+        raise KernelError(f"{act}: expected a dense tensor")
+    out = torch.empty_like(x)
+    _call(_fn("ti_pointwise_act", [P, P, L, I, I, P]), _ptr(x), _ptr(out), x.numel(), POINTWISE_ACTS[act], _code(x, act), _stream())
+    return out
+
+
 def relu2(x: torch.Tensor) -> torch.Tensor:
     """max(x, 0)^2, elementwise."""
-    _need_cuda(x, what="relu2")
-    if not x.is_contiguous():
-        raise KernelError("relu2: expected a dense tensor")
-    out = torch.empty_like(x)
-    _call(_fn("ti_relu2", [P, P, L, I, P]), _ptr(x), _ptr(out), x.numel(), _code(x, "relu2"), _stream())
-    return out
+    return pointwise_act(x, "relu2")
 
 
 def route_by_table(ids: torch.Tensor, table: torch.Tensor, n_experts: int):
@@ -123,25 +133,28 @@ def experts_ffn(x: torch.Tensor, perm: torch.Tensor, off: torch.Tensor, w_gate_u
     return out
 
 
-def route_softmax(z: torch.Tensor, correction, n_experts: int, top: int, n_groups: int = 0, keep: int = 0, scale: float = 1.0):
+def route_softmax(z: torch.Tensor, correction, n_experts: int, top: int, n_groups: int = 0, keep: int = 0, scale: float = 1.0,
+                  logit_bias=None):
     """z float32 [M, >= experts] (rows may be strided) -> (perm int32 [M * top], off int32 [experts + 1], weight float32
     [M * top]): with s = softmax(z) over the experts, every token's ``top`` experts by s + correction (float32 [experts] or
     None), chosen only among the ``keep`` best of ``n_groups`` equal runs of neighbouring experts (a run's score: its
-    largest s + correction; ``n_groups`` <= 1: no runs); a pair's weight is its s over the sum of the token's chosen s, times
+    largest s + correction; ``n_groups`` <= 1: no runs; without a correction the choice is by the logits themselves);
+    ``logit_bias`` (float32 [experts] or None) is added to the logits before anything else; a pair's weight is its s over the sum of the token's chosen s, times
     ``scale``.  The pairs come out grouped by expert (csrc/moe_router.cu)."""
-    _need_cuda(z, correction, what="moe_route_softmax")
+    _need_cuda(z, correction, logit_bias, what="moe_route_softmax")
     if z.dtype != torch.float32 or z.dim() != 2 or z.stride(1) != 1 or z.shape[1] < n_experts:
         raise KernelError("moe_route_softmax: the router's logits must be float32 [tokens, experts] with dense rows")
-    if correction is not None and (correction.dtype != torch.float32 or tuple(correction.shape) != (n_experts,) or not correction.is_contiguous()):
-        raise KernelError("moe_route_softmax: the correction must be dense float32 [experts]")
+    for t in (correction, logit_bias):
+        if t is not None and (t.dtype != torch.float32 or tuple(t.shape) != (n_experts,) or not t.is_contiguous()):
+            raise KernelError("moe_route_softmax: the correction and the logits' bias must be dense float32 [experts]")
     M = z.shape[0]
     dev = z.device
     perm = torch.empty(M * top, dtype=torch.int32, device=dev)
     off = torch.empty(n_experts + 1, dtype=torch.int32, device=dev)
     scratch = torch.empty(M * top, dtype=torch.int32, device=dev)
     weight = torch.empty(M * top, dtype=torch.float32, device=dev)
-    _call(_fn("ti_moe_route_softmax", [P, L, P, I, I, I, I, F, I, P, P, P, P, P]), _ptr(z), z.stride(0), _ptr(correction), int(n_experts),
-          int(top), int(n_groups), int(keep), float(scale), M, _ptr(perm), _ptr(off), _ptr(scratch), _ptr(weight), _stream())
+    _call(_fn("ti_moe_route_softmax", [P, L, P, P, I, I, I, I, F, I, P, P, P, P, P]), _ptr(z), z.stride(0), _ptr(logit_bias), _ptr(correction),
+          int(n_experts), int(top), int(n_groups), int(keep), float(scale), M, _ptr(perm), _ptr(off), _ptr(scratch), _ptr(weight), _stream())
     return perm, off, weight
 
 

@@ -85,10 +85,13 @@ def rglru_scan(gates: torch.Tensor, u: torch.Tensor, z: torch.Tensor, gate_bias_
 
 
 def delta_rule(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, decay_logit: torch.Tensor, dt_bias: torch.Tensor,
-               rate: torch.Tensor, beta_logit: torch.Tensor, state: torch.Tensor, state_offset: int, batch) -> torch.Tensor:
-    """q, k [M, qk_heads, dim] and v [M, heads, vdim] after their convolutions (not yet unit vectors); decay_logit float32
-    [M, heads * dim]; dt_bias float32 [heads * dim]; rate float32 [heads]; beta_logit [M, heads].  Returns float32
-    [M, heads * vdim]; the state [heads, dim, vdim] per slot is left as it is after the step's tokens."""
+               rate: torch.Tensor, beta_logit: torch.Tensor, state: torch.Tensor, state_offset: int, batch,
+               head_decay: bool = False) -> torch.Tensor:
+    """q, k [M, qk_heads, dim] and v [M, heads, vdim] after their convolutions (not yet unit vectors); a decay per key
+    channel: decay_logit float32 [M, heads * dim], dt_bias float32 [heads * dim]; with ``head_decay`` one per head:
+    decay_logit [M, heads] of the tokens' type (rows may be strided), dt_bias float32 [heads]; rate float32 [heads];
+    beta_logit [M, heads].  Returns float32 [M, heads * vdim]; the state [heads, dim, vdim] per slot is left as it is after
+    the step's tokens."""
     _need_cuda(q, k, v, decay_logit, dt_bias, rate, beta_logit, state, what="delta_rule")
     M, G, dim = q.shape
     H, vdim = v.shape[1], v.shape[2]
@@ -97,20 +100,22 @@ def delta_rule(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, decay_logit: t
     for t in (q, k, v):
         if t.stride(2) != 1 or t.stride(1) != t.shape[2]:
             raise KernelError("delta_rule: heads of a token must be dense")
-    if decay_logit.dtype != torch.float32 or tuple(decay_logit.shape) != (M, H * dim) or not decay_logit.is_contiguous():
-        raise KernelError(f"delta_rule: the decay logits must be dense float32 [{M}, {H * dim}]")
+    n_decay = H if head_decay else H * dim
+    if decay_logit.dtype != (q.dtype if head_decay else torch.float32) or tuple(decay_logit.shape) != (M, n_decay) or decay_logit.stride(1) != 1:
+        raise KernelError(f"delta_rule: the decay logits must be [{M}, {n_decay}] with dense rows, "
+                          f"{'of the type of the tokens' if head_decay else 'float32'}")
     if tuple(beta_logit.shape) != (M, H) or beta_logit.dtype != q.dtype or beta_logit.stride(1) != 1:
         raise KernelError("delta_rule: the write-strength logits must be [tokens, heads] of the tokens' type")
-    _vec(dt_bias, H * dim, "delta_rule: the decay bias")
+    _vec(dt_bias, n_decay, "delta_rule: the decay bias")
     _vec(rate, H, "delta_rule: the rates")
     base, stride = _state_part(state, state_offset, H * dim * vdim, "delta_rule")
     o = torch.zeros((M, H * vdim), dtype=torch.float32, device=q.device)
     # unit queries and keys, decays and betas of all tokens, made by a kernel of their own before the recurrence
-    scratch = torch.empty(M * (2 * G * dim + H * dim + H), dtype=torch.float32, device=q.device)
-    _call(_fn("ti_delta_rule_scan", [P, P, P, L, L, L, P, P, P, P, L, P, P, L, P, P, P, I, I, I, I, I, I, I, P]),
-          _ptr(q), _ptr(k), _ptr(v), q.stride(0), k.stride(0), v.stride(0), _ptr(decay_logit), _ptr(dt_bias), _ptr(rate),
-          _ptr(beta_logit), beta_logit.stride(0), _ptr(o), base, stride, _ptr(scratch), _ptr(batch.cu_new), _ptr(batch.seq_slot),
-          batch.n_seq, M, H, G, dim, vdim, _code(q, "delta_rule"), _stream(), launches=2)
+    scratch = torch.empty(M * (2 * G * dim + n_decay + H), dtype=torch.float32, device=q.device)
+    _call(_fn("ti_delta_rule_scan", [P, P, P, L, L, L, P, L, I, P, P, P, L, P, P, L, P, P, P, I, I, I, I, I, I, I, P]),
+          _ptr(q), _ptr(k), _ptr(v), q.stride(0), k.stride(0), v.stride(0), _ptr(decay_logit), decay_logit.stride(0), 1 if head_decay else 0,
+          _ptr(dt_bias), _ptr(rate), _ptr(beta_logit), beta_logit.stride(0), _ptr(o), base, stride, _ptr(scratch), _ptr(batch.cu_new),
+          _ptr(batch.seq_slot), batch.n_seq, M, H, G, dim, vdim, _code(q, "delta_rule"), _stream(), launches=2)
     return o
 
 

@@ -211,6 +211,11 @@ class Head(Part):
 class Block(Part):
     mixer: Mixer
 
+    def memory_request(self):
+        """What the cache keeps for the layer: the mixer's request, unless the block carries something of its own beside it
+        (then a tuple, whose views ``forward`` takes apart)."""
+        return self.mixer.memory_request()
+
     def launch_plan(self, n_seq: int, plan_len: int, dtype, device, n_live=None):
         """As Mixer.launch_plan, for the whole block."""
         return self.mixer.launch_plan(n_seq, plan_len, dtype, device, n_live)

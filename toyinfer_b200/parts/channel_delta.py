@@ -103,8 +103,8 @@ class ChannelDeltaAttention(Mixer):
         self.w_o = t("o").contiguous()
 
     def check_kernels(self, dtype) -> None:
-        if self.dim > 128:
-            raise K.KernelError(f"delta rule: heads of {self.dim} query/key elements are not supported (up to 128)")
+        if self.dim > 256:
+            raise K.KernelError(f"delta rule: heads of {self.dim} query/key elements are not supported (up to 256)")
         if self.taps > 8:
             raise K.KernelError(f"short convolution: {self.taps} taps are not supported (up to 8)")
 

@@ -1,4 +1,4 @@
-"""Multi-head latent attention with a sliding window and per-head sinks.
+"""Multi-head latent attention, with a sliding window and per-head sinks where a design has them.
 
 Per token x: q = Wq x, head by head [``dim`` plain | ``rot_dim`` rotated]; d = Wdkv x;
 c = rms(d[:kv_rank]) * w (the latent), r = rotate(d[kv_rank:]) (one rotated key part for all
@@ -10,6 +10,10 @@ The cache keeps [c | r] per position, one row for all heads (a request without v
 value is read out of the same row).  The kernels never form keys or values per head: the
 query is carried through Wuk into the latent space, the attention runs over the cached rows,
 and the result goes through Wuv (kernels/latent.py).  q and d come from one product.
+
+The kernels turn elements (e, e + rot / 2) of a rotated part together.  A position encoding that pairs neighbours
+(2e, 2e + 1) is met when weights are bound: the rows that make the rotated parts of q and of the key are put in the order
+0, 2, 4, ..., 1, 3, 5, ...  Scores are sums over the rotated part, so an order that query and key share changes nothing.
 """
 from __future__ import annotations
 
@@ -46,8 +50,6 @@ class LatentAttention(Mixer):
         if self.rot:
             try:
                 self.pos = ctx.positions[position]
-                if getattr(self.pos, "pairing", "half") != "half":
-                    raise ValueError(f"attention at {prefix!r}: its kernels turn elements (e, e + rot / 2) together, the position encoding {position!r} pairs neighbours")
             except KeyError:
                 raise ValueError(f"latent attention at {prefix!r} names unknown position encoding {position!r}") from None
             tables = getattr(self.pos, "dim", None)
@@ -70,7 +72,14 @@ class LatentAttention(Mixer):
         return s
 
     def bind(self, tensors: Dict[str, torch.Tensor]) -> None:
-        self.w_qd = torch.cat([tensors.pop(self.names["q"]), tensors.pop(self.names["dkv"])], dim=0).contiguous()
+        w_q, w_d = tensors.pop(self.names["q"]), tensors.pop(self.names["dkv"])
+        if self.pos is not None and getattr(self.pos, "pairing", "half") == "neighbours":
+            first, second = torch.arange(0, self.rot, 2), torch.arange(1, self.rot, 2)
+            order = torch.cat([first, second])
+            head = torch.cat([torch.arange(self.dim), self.dim + order]).to(w_q.device)
+            w_q = w_q.view(self.n_heads, self.dim + self.rot, self.hidden)[:, head].reshape(-1, self.hidden)
+            w_d = w_d[torch.cat([torch.arange(self.rank), self.rank + order]).to(w_d.device)]
+        self.w_qd = torch.cat([w_q, w_d], dim=0).contiguous()
         self.w_uk = tensors.pop(self.names["uk"]).contiguous()
         self.w_uv = tensors.pop(self.names["uv"]).contiguous()
         self.w_o = tensors.pop(self.names["o"]).contiguous()

@@ -92,13 +92,17 @@ class GatedDense(FeedForward):
         return K.linear(K.linear_swiglu(x, self.w_gate_up, self.act, self.limit), self.w_down)
 
 
-class SquaredReLU(FeedForward):
-    """y = Wdown relu(Wup x)^2; no gate, no bias."""
+class UngatedDense(FeedForward):
+    """y = Wdown act(Wup x) with ``act`` "relu2" (the squared ReLU) or "gelu" (by the error function); no gate, no bias."""
 
     captures_start = True
 
-    def __init__(self, ctx: BuildContext, prefix: str, intermediate_size: int, names: Optional[Dict[str, str]] = None):
+    def __init__(self, ctx: BuildContext, prefix: str, intermediate_size: int, act: str = "relu2", names: Optional[Dict[str, str]] = None):
+        from ..kernels.moe import POINTWISE_ACTS
+        if act not in POINTWISE_ACTS:
+            raise ValueError(f"feed-forward at {prefix!r}: unknown activation {act!r}; known: {sorted(POINTWISE_ACTS)}")
         self.hidden = ctx.hidden_size
+        self.act = act
         self.inter = int(intermediate_size)
         n = {"up": "up", "down": "down"}
         n.update(names or {})
@@ -115,7 +119,7 @@ class SquaredReLU(FeedForward):
 
     def forward(self, x, batch) -> torch.Tensor:
         from ..kernels import moe as KM
-        return K.linear(KM.relu2(K.linear(x, self.w_up)), self.w_down)
+        return K.linear(KM.pointwise_act(K.linear(x, self.w_up), self.act), self.w_down)
 
 
 class TableMoE(FeedForward):
@@ -169,7 +173,8 @@ class TableMoE(FeedForward):
 
 
 register_part("feed_forward", "gated_dense", GatedDense)
-register_part("feed_forward", "relu2", SquaredReLU)
+register_part("feed_forward", "relu2", UngatedDense)
+register_part("feed_forward", "ungated_dense", UngatedDense)
 register_part("feed_forward", "table_moe", TableMoE)
 
 
@@ -244,11 +249,11 @@ register_part("feed_forward", "scored_moe", ScoredMoE)
 
 
 class SoftmaxMoE(FeedForward):
-    """Mixture of silu-gated experts under a softmax router with a choice correction and expert groups: z = Wr x (float32),
-    s = softmax(z) over all experts; experts are CHOSEN by s + correction (a stored value per expert), only among the
+    """Mixture of silu-gated experts under a softmax router with a choice correction and expert groups: z = Wr x (float32;
+    with ``router_bias`` a stored value per expert is added), s = softmax(z) over all experts; experts are CHOSEN by s + correction (a stored value per expert), only among the
     experts of the ``keep`` best of ``n_groups`` equal runs of neighbouring experts (a run's score is its largest choice
     score); the ``top`` chosen experts' outputs are weighted by their s, divided by the sum of the chosen s, times
-    ``scale``.  An expert: Wdown (silu(Wgate x) * (Wup x)); a shared expert of the same form (its own width) may run for
+    ``scale``.  (Without a correction and with a scale of 1 that is: the largest logits, under a softmax over them alone.)  An expert: Wdown (silu(Wgate x) * (Wup x)); a shared expert of the same form (its own width) may run for
     every token and is added as it is.  No biases.  The step's (token, choice) pairs are grouped by expert on the device
     and every product runs once over all groups (kernels/moe.py)."""
 
@@ -256,9 +261,10 @@ class SoftmaxMoE(FeedForward):
 
     def __init__(self, ctx: BuildContext, prefix: str, n_experts: int, top: int, intermediate_size: int, n_groups: int = 0,
                  keep: int = 0, scale: float = 1.0, correction: bool = True, shared_size: int = 0,
-                 names: Optional[Dict[str, str]] = None):
+                 router_bias: bool = False, names: Optional[Dict[str, str]] = None):
         self.hidden = ctx.hidden_size
         self.n_experts, self.top, self.inter, self.shared = int(n_experts), int(top), int(intermediate_size), int(shared_size)
+        self.biased = bool(router_bias)
         self.n_groups, self.keep, self.scale, self.corrected = int(n_groups), int(keep), float(scale), bool(correction)
         if not (1 <= self.top <= self.n_experts):
             raise ValueError(f"moe at {prefix!r}: {self.top} of {self.n_experts} experts per token")
@@ -266,11 +272,11 @@ class SoftmaxMoE(FeedForward):
                                   or self.keep * (self.n_experts // self.n_groups) < self.top):
             raise ValueError(f"moe at {prefix!r}: {self.n_experts} experts in {self.n_groups} groups of which {self.keep} stay, "
                              f"{self.top} per token")
-        n = {"expert": "e{}.", "gate": "gate", "up": "up", "down": "down", "router": "router", "correction": "correction",
-             "shared": "shared."}
+        n = {"expert": "e{}.", "gate": "gate", "up": "up", "down": "down", "router": "router", "router_bias": "router.b",
+             "correction": "correction", "shared": "shared."}
         n.update(names or {})
         self.prefix, self.n = prefix, n
-        self.w_gate_up = self.w_down = self.w_router = self.correction = self.ws_gate_up = self.ws_down = None
+        self.w_gate_up = self.w_down = self.w_router = self.b_router = self.correction = self.ws_gate_up = self.ws_down = None
 
     def _name(self, e: int, which: str) -> str:
         return self.prefix + self.n["expert"].format(e) + self.n[which]
@@ -282,6 +288,8 @@ class SoftmaxMoE(FeedForward):
             s[self._name(e, "up")] = ParamSpec((self.inter, self.hidden), std=0.05)
             s[self._name(e, "down")] = ParamSpec((self.hidden, self.inter), std=0.05)
         s[self.prefix + self.n["router"]] = ParamSpec((self.n_experts, self.hidden), std=0.3)
+        if self.biased:
+            s[self.prefix + self.n["router_bias"]] = ParamSpec((self.n_experts,), role="norm", init="normal", std=0.3)
         if self.corrected:
             s[self.prefix + self.n["correction"]] = ParamSpec((self.n_experts,), role="norm", init="normal", std=0.05)
         if self.shared:
@@ -304,6 +312,8 @@ class SoftmaxMoE(FeedForward):
                                       for e in E]).contiguous()
         self.w_down = torch.stack([tensors.pop(self._name(e, "down")) for e in E]).contiguous()
         self.w_router = tensors.pop(self.prefix + self.n["router"]).contiguous()
+        if self.biased:
+            self.b_router = tensors.pop(self.prefix + self.n["router_bias"]).to(torch.float32).contiguous()
         if self.corrected:
             self.correction = tensors.pop(self.prefix + self.n["correction"]).to(torch.float32).contiguous()
         if self.shared:
@@ -316,7 +326,7 @@ class SoftmaxMoE(FeedForward):
         from ..kernels import moe as KM
         M = x.shape[0]
         z = K.linear(x, self.w_router, out_dtype=torch.float32)
-        perm, off, weight = KM.route_softmax(z, self.correction, self.n_experts, self.top, self.n_groups, self.keep, self.scale)
+        perm, off, weight = KM.route_softmax(z, self.correction, self.n_experts, self.top, self.n_groups, self.keep, self.scale, self.b_router)
         y, place, _ = KM.expert_pairs(x, perm, off, self.w_gate_up, self.w_down, self.top, float("inf"), 1.0, 0.0)
         shared = K.linear(K.linear_swiglu(x, self.ws_gate_up, "silu"), self.ws_down) if self.shared else None
         return KM.combine_gated(y, place, weight, shared, None, M, self.top)

@@ -130,7 +130,7 @@ class DecoderModel(Part):
         """One request (or None) per schedule entry; a borrowing entry asks for nothing."""
         out = []
         for e in self.schedule:
-            out.append(None if e.memory_of is not None else self.blocks[e.layer].mixer.memory_request())
+            out.append(None if e.memory_of is not None else self.blocks[e.layer].memory_request())
         return out
 
     def launch_plan(self, n_seq: int, plan_len: int, n_live: Optional[int] = None):

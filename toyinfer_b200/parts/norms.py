@@ -146,3 +146,38 @@ class WideScalarRMSNorm(Norm):
 
 
 register_part("norm", "wide_scalar_rmsnorm", WideScalarRMSNorm)
+
+
+class DepthRMSNorm(Norm):
+    """The norm that reads a float32 stream averaged over depth (kernels/depth.py): the pending layer's result is formed and
+    written, the average over the embedding and all results is taken, normed, and, where the reader asks for it, shifted by
+    a token, in one kernel.  The weight is float32 whatever the engine's type; the normed rows come out in the engine's
+    type."""
+
+    def __init__(self, ctx: BuildContext, prefix: str, size: int, eps: float, name: str = "weight"):
+        self.size, self.eps = int(size), float(eps)
+        self.weight_name = prefix + name
+        self.weight: Optional[torch.Tensor] = None
+        self.out_dtype = ctx.dtype
+
+    def param_specs(self) -> Dict[str, ParamSpec]:
+        return {self.weight_name: ParamSpec((self.size,), role="norm", init="one_plus_normal", std=0.1)}
+
+    def bind(self, tensors: Dict[str, torch.Tensor]) -> None:
+        self.weight = tensors.pop(self.weight_name).to(torch.float32).contiguous()
+
+    def read_forward(self, x0: torch.Tensor, pending, shift=None):
+        """(normed rows, shifted normed rows or None, the history with the pending layer's result); ``pending`` is a
+        kernels.depth.DepthUpdate or None, ``shift`` a kernels.depth.ShiftedRead or None."""
+        from ..kernels import depth
+        return depth.depth_norm(x0, pending, self.weight, self.eps, self.out_dtype, shift)[:3]
+
+    def forward(self, x: torch.Tensor) -> torch.Tensor:
+        return self.read_forward(x, None)[0]
+
+    def gather_add_forward(self, h: torch.Tensor, delta, rows: torch.Tensor) -> torch.Tensor:
+        from ..kernels import depth
+        return depth.depth_norm(h, delta, self.weight, self.eps, self.out_dtype, rows=rows)[0]
+
+
+register_part("norm", "depth_rmsnorm", DepthRMSNorm)

@@ -56,12 +56,15 @@ def banded_frequencies(dim: int, theta: float, factor: float, original: int, low
 
 def rotary_tables(dim: int, theta: float, max_positions: int, scaling: Optional[dict] = None) -> Tuple[torch.Tensor, torch.Tensor]:
     """cos and sin of pos * f_i with f_i = theta^(-2i/dim) (or the blended frequencies and magnitude of ``scaling``:
-    factor, original, fast, slow; or, with ``kind`` "bands", the banded frequencies of factor, original, low, high),
-    computed in 64-bit, returned as float32."""
+    factor, original, fast, slow; or, with ``kind`` "bands", the banded frequencies of factor, original, low, high; or, with
+    ``kind`` "linear", every frequency over factor), computed in 64-bit, returned as float32."""
     half = dim // 2
     if scaling and scaling.get("kind") == "bands":
         inv_freq, magnitude = banded_frequencies(dim, float(theta), float(scaling["factor"]), int(scaling["original"]),
                                                  float(scaling["low"]), float(scaling["high"])), 1.0
+    elif scaling and scaling.get("kind") == "linear":
+        i = torch.arange(half, dtype=torch.float64)
+        inv_freq, magnitude = torch.pow(torch.tensor(float(theta), dtype=torch.float64), -(2.0 * i) / dim) / float(scaling["factor"]), 1.0
     elif scaling:
         inv_freq, magnitude = blended_frequencies(dim, float(theta), float(scaling["factor"]), int(scaling["original"]),
                                                   float(scaling["fast"]), float(scaling["slow"]))
@@ -75,7 +78,7 @@ def rotary_tables(dim: int, theta: float, max_positions: int, scaling: Optional[
 
 class RotaryHalf(PositionEncoding):
     """``scaling``: None, or the stretch for long contexts (see blended_frequencies; with ``kind`` "bands" see
-    banded_frequencies).  ``max_positions`` is the
+    banded_frequencies; with ``kind`` "linear" every frequency is divided by ``factor``).  ``max_positions`` is the
     most the tables may ever hold; with ``lazy`` they are built for as many positions as ``ensure`` is told (the
     engine says how long its sequences get before the first step), not for the model's nominal limit."""
 
@@ -91,12 +94,12 @@ class RotaryHalf(PositionEncoding):
         self.max_positions = int(max_positions)
         self.scaling = dict(scaling) if scaling else None
         if self.scaling:
-            bands = self.scaling.get("kind") == "bands"
-            keys = ("factor", "original", "low", "high") if bands else ("factor", "original", "fast", "slow")
+            kind = self.scaling.get("kind")
+            keys = {"bands": ("factor", "original", "low", "high"), "linear": ("factor",)}.get(kind, ("factor", "original", "fast", "slow"))
             for key in keys:
                 if key not in self.scaling:
                     raise ValueError(f"rotary scaling needs {key!r}")
-            if not all(self.scaling[key] > 0 for key in keys) or (not bands and self.scaling["factor"] < 1.0):
+            if not all(self.scaling[key] > 0 for key in keys) or (kind not in ("bands", "linear") and self.scaling["factor"] < 1.0):
                 raise ValueError(f"rotary scaling out of range: {self.scaling}")
         self.device = ctx.device
         self.cos = self.sin = None

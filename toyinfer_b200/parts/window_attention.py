@@ -21,7 +21,8 @@ of its own over the same values, a1 and a2; with lambda = exp(lq1 . lk1) - exp(l
 per head.  The gate's rows ride with the q, k, v projection.
 
 ``kept_window_attention`` (one map): biases on all four projections (each optional); every head of q and of k normed over
-its own elements with one weight [dim] for all heads; the first ``rot_dim`` elements of every head of q and k rotated by
+its own elements with one weight [dim] for all heads (``head_norm`` "unit": over its root mean square, without a weight; a
+rotation keeps a head's root mean square, so such a norm may as well stand after the rotation); the first ``rot_dim`` elements of every head of q and k rotated by
 the token's position, in the pairing that the position encoding names; key j is visible to the query at i when
 0 <= i - j < window, or when j <= i and j < keep_first: the first ``keep_first`` positions of a sequence stay visible to
 every later query, at their own positions; softmax over the visible keys.  Its result may be scaled and placed in the
@@ -209,12 +210,14 @@ class KeptWindowAttention(_WindowAttention):
 
     def __init__(self, ctx: BuildContext, prefix: str, n_heads: int, n_kv_heads: int, dim: int, vdim: int, scale: float,
                  window: int, eps: float, keep_first: int = 0, position: Optional[str] = None, biases: bool = True,
-                 head_norm: bool = True, names: Optional[Dict[str, str]] = None):
+                 head_norm=True, names: Optional[Dict[str, str]] = None):
         self._sizes(ctx, prefix, n_heads, n_kv_heads, dim, vdim, scale, window, eps)
         if int(keep_first) < 0:
             raise ValueError(f"attention at {prefix!r}: {keep_first} kept first positions")
         self.keep_first = int(keep_first) if self.window > 0 else 0
-        self.biases, self.head_norm = bool(biases), bool(head_norm)
+        if head_norm not in (True, False, "unit"):
+            raise ValueError(f"attention at {prefix!r}: head_norm is True, False or 'unit', got {head_norm!r}")
+        self.biases, self.head_norm = bool(biases), head_norm
         self.position = None
         if position is not None:
             if position not in ctx.positions:
@@ -244,7 +247,7 @@ class KeptWindowAttention(_WindowAttention):
         if self.biases:
             for k, rows in (("q", H * d), ("k", G * d), ("v", G * vd), ("o", self.hidden)):
                 s[self._name(k, True)] = small((rows,), init="normal", std=0.1)
-        if self.head_norm:
+        if self.head_norm is True:
             s[self._name("q_norm")] = small((d,), init="one_plus_normal", std=0.1)
             s[self._name("k_norm")] = small((d,), init="one_plus_normal", std=0.1)
         return s
@@ -257,7 +260,9 @@ class KeptWindowAttention(_WindowAttention):
         if self.biases:
             self.b_qkv = torch.cat([f32(self._name(k, True)) for k in ("q", "k", "v")]).contiguous()
             self.b_o = f32(self._name("o", True))
-        if self.head_norm:
+        if self.head_norm == "unit":
+            self.q_w = self.k_w = torch.ones(self.dim, dtype=torch.float32, device=self.w_o.device)
+        elif self.head_norm:
             self.q_w, self.k_w = f32(self._name("q_norm")), f32(self._name("k_norm"))
 
     def launch_plan(self, n_seq: int, plan_len: int, dtype, device, n_live=None):
