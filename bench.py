@@ -18,7 +18,7 @@ error of the logits of a 512-token prompt's last place and of 8 decoded places.
 Every decode step reads all weights (8 GB) and the live sequences' cache, far more than
 the 126 MB L2, so nothing is flushed between steps.
 
-``--design kadodra`` (or ``tusasun``, ``bagasun``, ``bolisun``) measures another design instead (see run_design): prompt and decode rates and
+``--design kadodra`` (or ``tusasun``, ``bagasun``, ``bolisun``, ``mikipel``) measures another design instead (see run_design): prompt and decode rates and
 the device time of every stage of a layer at real layer sizes, beside the dense model at equal size.
 """
 from __future__ import annotations
@@ -531,6 +531,25 @@ def _bolisun_config(width, heads, layers, kind, vocab=32000):
             "layers": [json.loads(json.dumps(layer)) for _ in range(layers)], "max_positions": 8192}
 
 
+def _mikipel_config(width, heads, layers, kind, vocab=32000):
+    """``layers`` equal layers over a depth-averaged float32 stream, a token-shifted mixer beside its feed-forward: "attention" (heads
+    of 128, 4 query heads per kv head, whole heads rotated; a gelu feed-forward of 4 width), "latent" (the sizes of Kadodra's
+    latent attention, without a window; the same feed-forward) or "delta" (gated delta rule, a decay per head, heads of 128;
+    sixteen silu-gated experts of the model's width, two per token)."""
+    dense = {"kind": "dense", "ff": 4 * width}
+    if kind == "attention":
+        layer = {"type": "attention", "mixer": {"heads": heads, "kv_heads": max(1, heads // 4), "dim": 128, "vdim": 128, "scale": 128 ** -0.5,
+                                                "rot": {"base": 1e6, "dims": 128, "scaling": {"factor": 4.0}}}, "mlp": dense}
+    elif kind == "latent":
+        layer = {"type": "latent_attention", "mixer": {"heads": heads, "dim": 64, "rot_dim": 64, "vdim": 128, "kv_rank": 512,
+                                                       "scale": 128 ** -0.5, "rot": {"base": 1e6, "dims": 64}}, "mlp": dense}
+    else:
+        layer = {"type": "delta", "mixer": {"heads": heads, "kv_heads": heads, "dim": 128, "vdim": 128, "conv": 4},
+                 "mlp": {"kind": "moe", "expert": {"ff": width}, "router": {"experts": 16, "top": 2}}}
+    return {"architecture": "Mikipel", "vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "embedding": {"scale": 1.0}, "residual_mult": 0.7,
+            "logit_softcap": 30.0, "layers": [json.loads(json.dumps(layer)) for _ in range(layers)], "max_positions": 8192}
+
+
 def _qwen3_like(width, heads, layers, vocab=32000):
     """The dense model of the same width, head count and layers; its three feed-forward matrices of 8/3 width hold what the
     other design's two of 4 width (or its two active experts of three matrices each, 6 width... the nearest round size) hold."""
@@ -547,14 +566,22 @@ def run_design(name: str, widths, layers: int, tokens: int, batch: int, context:
     import torch
     from toyinfer_b200.engine import Engine
     from toyinfer_b200.tracing import Tracer
-    if name not in ("kadodra", "tusasun", "bagasun", "bolisun"):
-        raise SystemExit(f"bench.py: unknown design {name!r} (kadodra, tusasun, bagasun, bolisun)")
+    if name not in ("kadodra", "tusasun", "bagasun", "bolisun", "mikipel"):
+        raise SystemExit(f"bench.py: unknown design {name!r} (kadodra, tusasun, bagasun, bolisun, mikipel)")
     for width in widths:
         heads = width // 128
         if name == "kadodra":
             models = [("kadodra latent+dense", _kadodra_config(width, heads, layers, "latent")),
                       ("kadodra lightning+experts", _kadodra_config(width, heads, layers, "lightning")),
                       ("qwen3 dense", _qwen3_like(width, heads, layers))]
+        elif name == "mikipel":     # the parallel layer and the latent rows are Kadodra's, the delta rule Tusasun's, the attention the dense model's
+            models = [("mikipel attention+dense", _mikipel_config(width, heads, layers, "attention")),
+                      ("qwen3 dense", _qwen3_like(width, heads, layers)),
+                      ("mikipel latent+dense", _mikipel_config(width, heads, layers, "latent")),
+                      ("kadodra latent+dense", _kadodra_config(width, heads, layers, "latent")),
+                      ("mikipel delta+experts", _mikipel_config(width, heads, layers, "delta")),
+                      ("tusasun delta+experts", _tusasun_config(width, heads, layers, "delta")),
+                      ("kadodra lightning+experts", _kadodra_config(width, heads, layers, "lightning"))]
         elif name == "bolisun":     # streams, attention and experts are Tusasun's; the decayed state is lightning's; the window Bagasun's
             models = [("bolisun window+retention, dense", _bolisun_config(width, heads, layers, "dense")),
                       ("bolisun window+retention, experts", _bolisun_config(width, heads, layers, "experts")),
@@ -657,6 +684,10 @@ def run_kernel(name: str, reps: int, eager: bool = False):
 
     def rnd(*shape, scale=1.0):
         return (torch.randn(*shape, generator=g, device=dev) * scale).to(torch.bfloat16)
+
+    def numbers(*defaults):                               # the case's numbers after the colon, defaults for those left out
+        given = [int(v) for v in name.split(":")[1].split(",")] if ":" in name else []
+        return given + list(defaults[len(given):])
 
     def make():
         if name.startswith("gemm:"):                     # gemm:M,N,K or gemm:M,N,K,BN,SPLITS (tile width and splits forced)
@@ -839,6 +870,41 @@ def run_kernel(name: str, reps: int, eager: bool = False):
             # x, B, C and the step sizes read, y written in float32; 2 multiply-adds per state element and token
             return (lambda: KR.ssd_scan(xbc, dt, dt_bias, rate, skip, heads, groups, N, vd, state, 0, batch)), \
                 xbc.numel() * 2 + dt.numel() * 2 + T * inner * 4, 4.0 * T * inner * N
+        if name.startswith("depth_norm"):                 # depth_norm[:TOKENS[,RESULTS[,WIDTH]]]: a layer boundary of a depth-averaged stream
+            from toyinfer_b200.kernels import depth
+            T, n, W = numbers(PREFILL_TOKENS, 3, 2048)
+            f32 = lambda *shape: torch.rand(*shape, generator=g, device=dev)
+            results = [f32(T, W) for _ in range(n)]
+            a, f, w, mix, state = rnd(T, W), rnd(T, W), f32(W), f32(W), torch.zeros(65 if T <= 64 else 2, W, device=dev)
+            pend = depth.DepthUpdate(results, a, f, 0.7, f32(n), f32(n + 1))
+            batch = fill_batch(BatchBuffers(T, T, dev), "extend", list(range(T)), [100] * T, [[0]] * T, T, 101) if T <= 64 \
+                else fill_batch(BatchBuffers(1, T, dev), "start", [0], [0], [[0] * T], 1, T)
+            shift = depth.ShiftedRead(mix, state, batch)
+            # the history and both outputs read; the result, the normed and the shifted row written
+            return (lambda: depth.depth_norm(results[0], pend, w, 1e-6, torch.bfloat16, shift)), T * W * (4 * n + 4 + 4 + 4), 0.0
+        if name.startswith("hyper_norm"):                 # hyper_norm[:TOKENS[,STREAMS[,WIDTH]]]: a sublayer boundary of several streams
+            from toyinfer_b200.kernels import hyper
+            T, n, W = numbers(PREFILL_TOKENS, 4, 2048)
+            f32 = lambda *shape: torch.rand(*shape, generator=g, device=dev)
+            X, y, w = f32(T, n * W), rnd(T, W), f32(W)
+            up = hyper.StreamUpdate(y, None, torch.eye(n, device=dev), f32(n))
+            read = f32(n)
+            return (lambda: hyper.hyper_norm(X, up, read, w, 1e-6, torch.bfloat16, n)), T * W * (8 * n + 2 + 2), 0.0
+        if name.startswith("delta_rule"):                 # delta_rule[:TOKENS[,head|channel[,HEADS]]]: the recurrence over one prompt (up to 64: single tokens)
+            from toyinfer_b200.kernels import recurrent as KR
+            opts = name.split(":")[1].split(",") if ":" in name else []
+            T, per_head, H_ = int(opts[0]) if opts else PREFILL_TOKENS, (opts[1] if len(opts) > 1 else "head") == "head", int(opts[2]) if len(opts) > 2 else 16
+            d = 128
+            f32 = lambda *shape: torch.rand(*shape, generator=g, device=dev)
+            q, k, v = rnd(T, H_, d), rnd(T, H_, d), rnd(T, H_, d)
+            decay = rnd(T, H_) if per_head else f32(T, H_ * d)
+            dt, rate, beta = f32(H_ if per_head else H_ * d) - 4.0, f32(H_) + 0.5, rnd(T, H_)
+            single = T <= 64
+            state = torch.zeros((T if single else 1) + 1, H_ * d * d, dtype=torch.float32, device=dev)
+            batch = fill_batch(BatchBuffers(T, T, dev), "extend", list(range(T)), [100] * T, [[0]] * T, T, 101) if single \
+                else fill_batch(BatchBuffers(1, T, dev), "start", [0], [0], [[0] * T], 1, T)
+            nb = T * H_ * d * (2 * 3 + 4) + (2 * T * H_ * d * d * 4 if single else 0)
+            return (lambda: KR.delta_rule(q, k, v, decay, dt, rate, beta, state, 0, batch, head_decay=per_head)), nb, 6.0 * T * H_ * d * d
         raise SystemExit(f"unknown kernel case {name!r}")
 
     fn, nbytes, flops = make()
@@ -892,13 +958,14 @@ def main() -> int:
                     "gemm_qkv, gemm_o, gemm_head, gemm_prefill, gemm:M,N,K[,BN,SPLITS], attn_decode[:BATCH,CONTEXT[,HEADS,KV_HEADS]], attn_decode_b64, attn_decode_b1, "
                     "attn_prefill[:TOKENS], attn_chunk[:CACHED,NEW[,HEAD_DIM]], add_rmsnorm[:TOKENS], rope_store[:TOKENS], "
                     "attn_window[:TOKENS[,sigmoid|diff|kept[,WINDOW[,cuda]]]], attn_window_prepare[:TOKENS[,sigmoid|diff|kept]], attn_window_decode[:BATCH,CONTEXT[,sigmoid|diff|kept[,WINDOW]]], "
-                    "ssd_scan[:TOKENS[,SEGMENT]], ssd_decode[:BATCH], mma_issue; "
+                    "ssd_scan[:TOKENS[,SEGMENT]], ssd_decode[:BATCH], depth_norm[:TOKENS[,RESULTS[,WIDTH]]], "
+                    "hyper_norm[:TOKENS[,STREAMS[,WIDTH]]], delta_rule[:TOKENS[,head|channel[,HEADS]]], mma_issue; "
                     "ref:all or ref:<case> times the reference's kernel recompiled for sm_100a beside this library's")
     ap.add_argument("--workload", default="", choices=["", "8b", "32b"],
                     help="run one of the larger described workloads end to end instead (8B or 32B shape)")
     ap.add_argument("--prompt-steps", default="", help="time one prompt step of each of these lengths instead (comma-separated), "
                     "with --layers layers")
-    ap.add_argument("--design", default="", help="measure another design beside its closest relations at equal size instead: kadodra, tusasun, bagasun or bolisun "
+    ap.add_argument("--design", default="", help="measure another design beside its closest relations at equal size instead: kadodra, tusasun, bagasun, bolisun or mikipel "
                     "(with --widths, --layers, --tokens, --batch, --context)")
     ap.add_argument("--widths", default="2048,4096", help="with --design: model widths (heads of 128)")
     ap.add_argument("--tokens", type=int, default=PREFILL_TOKENS, help="with --design: the prompt's tokens")

@@ -148,13 +148,13 @@ def delta_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, g: torch.Tenso
     G, d = q.shape[1], q.shape[2]
     S = torch.zeros(H, d, dv, dtype=F64) if S is None else S.clone()
     o = torch.zeros(T, H, dv, dtype=F64)
+    own = torch.arange(H) // (H // G)                   # the query/key head of every value head
     for t in range(T):
-        for h in range(H):
-            kk, qq = k[t, h // (H // G)], q[t, h // (H // G)]
-            M = g[t, h] * S[h]
-            u = beta[t, h] * (v[t, h] - M.T @ kk)
-            S[h] = M + torch.outer(kk, u)
-            o[t, h] = S[h].T @ qq
+        kk, qq = k[t, own], q[t, own]
+        M = g[t, :, None, None] * S
+        u = beta[t, :, None] * (v[t] - torch.einsum("hdv,hd->hv", M, kk))
+        S = M + kk[:, :, None] * u[:, None, :]
+        o[t] = torch.einsum("hdv,hd->hv", S, qq)
     return o, S
 
 
@@ -192,10 +192,14 @@ def route(t: torch.Tensor, top: int) -> Tuple[List[int], torch.Tensor]:
 def experts_ff(z: torch.Tensor, p: Dict[str, torch.Tensor], f: dict) -> torch.Tensor:
     logits = z @ p["router"].T + p["router.b"]
     out = torch.zeros(z.shape[0], p["e0.down"].shape[0], dtype=F64)
+    weight = torch.zeros_like(logits)                   # [T, experts], zero where an expert is not chosen
     for t in range(z.shape[0]):
         chosen, w = route(logits[t], int(f["router"]["top"]))
-        for e, we in zip(chosen, w):
-            out[t] += we * ((silu(p[f"e{e}.gate"] @ z[t]) * (p[f"e{e}.up"] @ z[t])) @ p[f"e{e}.down"].T)
+        weight[t, chosen] = w.to(F64)
+    for e in range(logits.shape[1]):
+        who = weight[:, e].nonzero()[:, 0]
+        zz = z[who]
+        out[who] += weight[who, e, None] * ((silu(zz @ p[f"e{e}.gate"].T) * (zz @ p[f"e{e}.up"].T)) @ p[f"e{e}.down"].T)
     return out
 
 
