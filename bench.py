@@ -890,6 +890,12 @@ def run_kernel(name: str, reps: int, eager: bool = False):
             up = hyper.StreamUpdate(y, None, torch.eye(n, device=dev), f32(n))
             read = f32(n)
             return (lambda: hyper.hyper_norm(X, up, read, w, 1e-6, torch.bfloat16, n)), T * W * (8 * n + 2 + 2), 0.0
+        if name.startswith("pointwise"):                  # pointwise[:TOKENS[,relu2|gelu[,FF]]]: an ungated feed-forward's activation
+            from toyinfer_b200.kernels import moe as KM
+            opts = name.split(":")[1].split(",") if ":" in name else []
+            T, act, ff = int(opts[0]) if opts else PREFILL_TOKENS, opts[1] if len(opts) > 1 else "gelu", int(opts[2]) if len(opts) > 2 else 8192
+            x = rnd(T, ff)
+            return (lambda: KM.pointwise_act(x, act)), 2 * T * ff * 2, 0.0
         if name.startswith("delta_rule"):                 # delta_rule[:TOKENS[,head|channel[,HEADS]]]: the recurrence over one prompt (up to 64: single tokens)
             from toyinfer_b200.kernels import recurrent as KR
             opts = name.split(":")[1].split(",") if ":" in name else []
@@ -959,7 +965,7 @@ def main() -> int:
                     "attn_prefill[:TOKENS], attn_chunk[:CACHED,NEW[,HEAD_DIM]], add_rmsnorm[:TOKENS], rope_store[:TOKENS], "
                     "attn_window[:TOKENS[,sigmoid|diff|kept[,WINDOW[,cuda]]]], attn_window_prepare[:TOKENS[,sigmoid|diff|kept]], attn_window_decode[:BATCH,CONTEXT[,sigmoid|diff|kept[,WINDOW]]], "
                     "ssd_scan[:TOKENS[,SEGMENT]], ssd_decode[:BATCH], depth_norm[:TOKENS[,RESULTS[,WIDTH]]], "
-                    "hyper_norm[:TOKENS[,STREAMS[,WIDTH]]], delta_rule[:TOKENS[,head|channel[,HEADS]]], mma_issue; "
+                    "hyper_norm[:TOKENS[,STREAMS[,WIDTH]]], delta_rule[:TOKENS[,head|channel[,HEADS]]], pointwise[:TOKENS[,relu2|gelu[,FF]]], mma_issue; "
                     "ref:all or ref:<case> times the reference's kernel recompiled for sm_100a beside this library's")
     ap.add_argument("--workload", default="", choices=["", "8b", "32b"],
                     help="run one of the larger described workloads end to end instead (8B or 32B shape)")

@@ -100,6 +100,7 @@ def test_feed_forward_on_its_own_stream_changes_nothing(folders, dtype):
         eng.step(list(zip(slots, ids)))
         got[two] = torch.cat([eng.step([(s, [(7 * t + i) % 200]) for i, s in enumerate(slots)]).clone() for t in range(12)])
         assert eng.graph_replays >= 10
+        assert all((b._side is not None) == (two and b.feed_forward is not None) for b in eng.model.blocks)
     assert torch.equal(got[True], got[False])
 
 

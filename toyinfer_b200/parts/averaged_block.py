@@ -25,6 +25,7 @@ from typing import Dict, Optional
 import torch
 
 from ..kernels.depth import DepthUpdate, MAX_RESULTS, ShiftedRead
+from ..tracing import ranged
 from .base import Block, BuildContext, ParamSpec, PartSpec, StateRequest, build_part, register_part
 
 
@@ -98,19 +99,14 @@ class AveragedParallelBlock(Block):
 
     def forward(self, h, delta, batch, mem, shared):
         trace = getattr(batch, "trace", None)
-        timed = trace is not None and trace.active
         mix_mem, before = self._memories(mem)
         read = ShiftedRead(self.shift, before.state, batch) if self.has_shift else None
         z, zs, results = self.norm.read_forward(h, delta, read)
         if zs is None:
             zs = z
-        ff = self.feed_forward
-        if timed:
-            with trace.range("layer.attn_block"):
-                a = self.mixer.forward(zs, batch, mix_mem, shared)
-            with trace.range("layer.mlp_block"):
-                f = ff.forward(z, batch) if ff is not None else None
-        elif ff is not None and self.two_streams and batch.mode == "extend" and z.is_cuda:
+        ff, f = self.feed_forward, None
+        beside = ff is not None and self.two_streams and batch.mode == "extend" and z.is_cuda and not (trace is not None and trace.timing)
+        if beside:
             # (memory: what the side stream made is used again on the side stream only, after a fork that follows its last reader)
             if self._side is None:
                 self._side = torch.cuda.Stream(device=z.device)
@@ -121,11 +117,13 @@ class AveragedParallelBlock(Block):
             with torch.cuda.stream(self._side):
                 f = ff.forward(z, batch)
                 joined.record(self._side)
+        with ranged(batch, "layer.attn_block"):
             a = self.mixer.forward(zs, batch, mix_mem, shared)
+        if beside:
             main.wait_event(joined)
-        else:
-            a = self.mixer.forward(zs, batch, mix_mem, shared)
-            f = ff.forward(z, batch) if ff is not None else None
+        elif ff is not None:
+            with ranged(batch, "layer.mlp_block"):
+                f = ff.forward(z, batch)
         # how the pending layer's y was formed is how this layer's input was formed
         c_in = delta.average_out if delta is not None else None
         return h, DepthUpdate(results, a, f, self.mult, c_in, self.average)
