@@ -358,6 +358,24 @@ def test_gelu_feed_forward(dtype, hidden, ff, M):
                                rtol=1e-2 if dtype == torch.bfloat16 else 1e-5, atol=1e-6)
 
 
+@pytest.mark.parametrize("act", ["gelu", "relu2"])
+@pytest.mark.parametrize("M,N,K", [(1, 200, 136), (1, 4096, 1024), (3, 77, 64), (8, 1000, 512), (16, 136, 264), (40, 512, 2048), (130, 264, 96),
+                                   (700, 1032, 520), (2100, 2048, 256), (256, 2560, 4096)])
+def test_activation_in_the_products_epilogue(act, M, N, K):
+    """Every product kernel (one token, few tokens, many tokens, a contraction cut into pieces) with the activation on its
+    32-bit results, against the activation of the exact product."""
+    import toyinfer_b200.kernels as TK
+    g = torch.Generator(device=DEV).manual_seed(M + N)
+    x = torch.randn(M, K, generator=g, device=DEV).to(torch.bfloat16)
+    w = (torch.randn(N, K, generator=g, device=DEV) * (2.5 / K ** 0.5)).to(torch.bfloat16)
+    before = TK.launch_count
+    got = TK.linear_act(x, w, act).double()
+    assert TK.launch_count == before + 1                 # no kernel of its own for the activation
+    z = x.double() @ w.double().T
+    want = plain.gelu(z) if act == "gelu" else torch.clamp(z, min=0.0) ** 2
+    torch.testing.assert_close(got, want, rtol=1e-2, atol=2e-4)
+
+
 def test_biased_router_against_the_rule():
     """The bias changes the choice and the weights; equal logits go to the lower index; logits so far below the largest that
     their softmax is zero are still chosen in their order."""

@@ -176,6 +176,25 @@ __device__ __forceinline__ float ti_gate_pair(float gate, float up, int kind, fl
     return up * ti_gate_act(gate, kind);
 }
 
+// Activations without a gate, applied value by value.  kind 4: the squared ReLU; kind 5: gelu by the error function,
+// z (1 + erf(z / sqrt(2))) / 2, exact in 32-bit.
+__device__ __forceinline__ float ti_pointwise(float z, int kind) {
+    if (kind == 4) { const float v = fmaxf(z, 0.f); return v * v; }
+    return 0.5f * z * (1.0f + erff(z * 0.70710678118654752f));
+}
+
+// The same for a result that is rounded to bfloat16: the complement of the error function by the rational-exponential
+// form 7.1.26 of Abramowitz and Stegun, "Handbook of Mathematical Functions" (absolute error of erf below 1.5e-7; its
+// exponential factor keeps gelu's left tail to within two steps of bfloat16 down to z = -6, where it has fallen to 1e-8).
+__device__ __forceinline__ float ti_pointwise_bf16(float z, int kind) {
+    if (kind == 4) { const float v = fmaxf(z, 0.f); return v * v; }
+    const float x = fabsf(z) * 0.70710678118654752f;
+    const float t = __fdividef(1.0f, fmaf(0.3275911f, x, 1.0f));
+    const float poly = fmaf(fmaf(fmaf(fmaf(1.061405429f, t, -1.453152027f), t, 1.421413741f), t, -0.284496736f), t, 0.254829592f) * t;
+    const float half = 0.5f * poly * __expf(-x * x);
+    return z * (z >= 0.f ? 1.0f - half : half);
+}
+
 template <typename F>
 static inline int ti_dispatch_dtype(int dtype, F&& f) {
     // f is called with a value of the element type

@@ -48,6 +48,7 @@ struct Args {
     long long ldx, ldw, ldo;
     int rows;       // weight rows per group, 8 to 16 (even for a gated product): see rows_per_group
     float gate_limit = 0.f;     // the limit of a gated product of kind 3 (ti_gate_pair)
+    int act = 0;                // 4 or 5: every value of an ungated product passes ti_pointwise_bf16
 };
 
 // NT: token tiles of 8 (1 or 2); WARPS per block; WPR: warps that share a group of 16 rows.
@@ -154,7 +155,8 @@ __global__ void __launch_bounds__(WARPS * 32, WARPS == 16 ? 2 : 3) skinny_kernel
                 const int in_group = g + (e >> 1) * 8;
                 const long long row = r0 + in_group;
                 const int tok = n * 8 + 2 * t + (e & 1);
-                if (in_group < R && row < a.N && tok < a.M) out[(size_t)tok * a.ldo + (size_t)row] = from_f32<OutT>(c[n][e]);
+                if (in_group < R && row < a.N && tok < a.M)
+                    out[(size_t)tok * a.ldo + (size_t)row] = from_f32<OutT>(a.act ? ti_pointwise_bf16(c[n][e], a.act) : c[n][e]);
             }
         }
     }
@@ -227,8 +229,8 @@ extern "C" void ti_set_skinny_rows(int rows) { g_force_rows = rows >= 8 && rows 
 
 // x[M, K] (row stride ldx), w[N, K] (row stride ldw), both bfloat16, M from 1 to 16; out[M, N]
 // bfloat16 or float32.  With `gated`, w's rows are (gate_0, up_0, gate_1, up_1, ...) and out is
-// [M, N / 2] = up * gate / (1 + exp(-gate)) in bfloat16.  K and the strides are multiples of 8
-// elements and the operands 16-byte aligned.  `sms`: the device's multiprocessors.  `late_start`:
+// [M, N / 2] = up * gate / (1 + exp(-gate)) in bfloat16 (codes 2 to 5 as for ti_linear_tc).  K and the strides are
+// multiples of 8 elements and the operands 16-byte aligned.  `sms`: the device's multiprocessors.  `late_start`:
 // see the note on launching at the top of this file.
 extern "C" int ti_linear_skinny(const void* x, const void* w, void* out, int M, int N, int K, long long ldx,
                                 long long ldw, long long ldo, int out_f32, int gated, float gate_limit, int sms, int late_start,
@@ -238,7 +240,8 @@ extern "C" int ti_linear_skinny(const void* x, const void* w, void* out, int M, 
     TI_REQUIRE(K % 8 == 0 && ldx % 8 == 0 && ldw % 8 == 0, "linear (small batch): K and the row strides must be multiples of 8 elements");
     TI_REQUIRE((reinterpret_cast<uintptr_t>(x) & 15) == 0 && (reinterpret_cast<uintptr_t>(w) & 15) == 0,
                "linear (small batch): operands must be 16-byte aligned");
-    TI_REQUIRE(!gated || (N % 2 == 0 && !out_f32), "linear (small batch): a gated product needs an even number of weight rows and a bfloat16 result");
+    TI_REQUIRE(gated >= 0 && gated <= 5, "linear (small batch): unknown activation %d", gated);
+    TI_REQUIRE(!gated || ((gated >= 4 || N % 2 == 0) && !out_f32), "linear (small batch): a gated product needs an even number of weight rows and a bfloat16 result");
     // Warps per row group, measured on the shapes of 4B- and 32B-sized layers: what counts is
     // how many warps have loads in flight, so a group's contraction is cut into 8 slices
     // whenever each slice keeps two steps, and into 16 (blocks of 16 warps, registers capped
@@ -251,6 +254,7 @@ extern "C" int ti_linear_skinny(const void* x, const void* w, void* out, int M, 
     if (wpr == 8 && groups * 8 < target && steps >= 16 * UNROLL) wpr = 16;
     Args a{(const bf16*)x, (const bf16*)w, out, M, N, K, ldx, ldw, ldo, 16};
     a.gate_limit = gate_limit;
+    if (gated >= 4) { a.act = gated; gated = 0; }
     return M <= 8 ? launch_nt<1>(a, out_f32, gated, wpr, sms, late_start != 0, stream)
                   : launch_nt<2>(a, out_f32, gated, wpr, sms, late_start != 0, stream);
 }

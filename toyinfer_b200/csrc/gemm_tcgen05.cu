@@ -240,7 +240,7 @@ extern "C" int ti_linear_tc_plan(int M, int N, int K, int sms, int* swap, int* b
 // x[M, K] (row stride ldx), w[N, K] (row stride ldw), both bfloat16; out[M, N] bfloat16 or
 // float32 with row stride ldo.  With `gated`, w's rows are (gate_0, up_0, gate_1, up_1, ...) and
 // out is [M, N / 2] = up * gate / (1 + exp(-gate)) (gated 1; 2: the tanh form of gelu; 3: the clamped pair of
-// ti_gate_pair with `gate_limit`).  `workspace` (float32) and `tickets` (int32, zero before the
+// ti_gate_pair with `gate_limit`; 4 and 5: no pairs, out is [M, N] with every value through ti_pointwise_bf16).  `workspace` (float32) and `tickets` (int32, zero before the
 // first use, left zero) as planned by ti_linear_tc_plan; tickets needs n_tiles entries and may be
 // null, in which case a second kernel adds the partial tiles of a split contraction, and the
 // many-token kernel deals out whole tiles only.
@@ -261,7 +261,8 @@ extern "C" int ti_linear_tc(const void* x, const void* w, void* out, int M, int 
     g.splits = splits; g.workspace = workspace; g.tickets = tickets;
     g.gated = gated; g.gate_limit = gate_limit;
     g.shared_tiles = p.walk && workspace && tickets ? p.shared : 0;      // without them: whole tiles only
-    TI_REQUIRE(!gated || (N % 2 == 0 && !out_f32), "linear (tcgen05): a gated product needs an even number of weight rows and a bfloat16 result");
+    TI_REQUIRE(gated >= 0 && gated <= 5, "linear (tcgen05): unknown activation %d", gated);
+    TI_REQUIRE(!gated || ((gated >= 4 || N % 2 == 0) && !out_f32), "linear (tcgen05): a gated product needs an even number of weight rows and a bfloat16 result");
     CUtensorMap am, bm;
     if (int rc = operand_map(swap ? w : x, g.rows_a, K, swap ? ldw : ldx, BM, &am)) return rc;
     // the other operand's box: a whole tile's rows; a pair's block loads half of them, or, where the

@@ -13,7 +13,7 @@ struct GemmArgs {
     int rows_a, rows_b, K;
     void* out; long long ld_out; int out_f32; int transposed;
     int splits; float* workspace; int* tickets;
-    int gated;      // rows of the weight operand come in (gate, up) pairs: store ti_gate_pair(gate, up), half as many columns (1: silu, 2: gelu, tanh form, 3: clamped)
+    int gated;      // rows of the weight operand come in (gate, up) pairs: store ti_gate_pair(gate, up), half as many columns (1: silu, 2: gelu, tanh form, 3: clamped); 4, 5: no pairs, every value passes ti_pointwise_bf16
     float gate_limit;   // the limit of kind 3
     int shared_tiles;   // many-token kernel: the first so many tiles are shared out by contraction steps (see TileWalk)
 };
@@ -28,7 +28,7 @@ __device__ __forceinline__ constexpr uint32_t instr_desc() {
 // All lanes of a warp must call it together (the gated, transposed form exchanges values
 // between neighbouring lanes).
 __device__ __forceinline__ void store_chunk(const GemmArgs& g, int i, int b0, int c, float (&r)[16], int lane) {
-    if (g.gated) {
+    if (g.gated && g.gated < 4) {
         // gate and up are neighbours along the weight operand's rows; both are rounded to
         // the storage type first, as if the product had been stored (src/decode.cu:756-762)
         if (g.transposed) {
@@ -66,6 +66,10 @@ __device__ __forceinline__ void store_chunk(const GemmArgs& g, int i, int b0, in
             }
         }
     } else if (i < g.rows_a) {
+        if (g.gated) {
+#pragma unroll
+            for (int e = 0; e < 16; e++) r[e] = ti_pointwise_bf16(r[e], g.gated);
+        }
         if (g.transposed) {
             // out[j, i]: the warp's lanes are consecutive i, so each j is one coalesced store
 #pragma unroll

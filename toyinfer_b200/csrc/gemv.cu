@@ -51,7 +51,7 @@ __device__ __forceinline__ void fma_piece(float (&acc)[M], const uint4& wv, cons
 template <int M, int R, int U, int WPR, int GATED, typename OutT>
 __global__ void __launch_bounds__(WARPS * 32)
 gemv_kernel(const bf16* x, const bf16* __restrict__ w, OutT* __restrict__ out, int N, int K,
-            long long ldx, long long ldw, long long ldo, float gate_limit) {
+            long long ldx, long long ldw, long long ldo, float gate_limit, int act) {
     ti_pdl_trigger();
     __shared__ float part_sum[WPR > 1 ? WARPS * R * M : 1];
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
@@ -124,7 +124,8 @@ gemv_kernel(const bf16* x, const bf16* __restrict__ w, OutT* __restrict__ out, i
         for (int r = 0; r < R; r++) {
             if (row0 + r >= N) break;
 #pragma unroll
-            for (int m = 0; m < M; m++) out[(size_t)m * ldo + (size_t)(row0 + r)] = from_f32<OutT>(acc[r][m]);
+            for (int m = 0; m < M; m++)
+                out[(size_t)m * ldo + (size_t)(row0 + r)] = from_f32<OutT>(act ? ti_pointwise_bf16(acc[r][m], act) : acc[r][m]);
         }
     }
 }
@@ -258,6 +259,7 @@ gemv_normed_kernel(const bf16* h, const bf16* delta, const NW* __restrict__ g, f
 struct Args {
     const bf16* x; const bf16* w; void* out; int N, K; long long ldx, ldw, ldo; cudaStream_t stream;
     float gate_limit = 0.f;     // the limit of a gated product of kind 3 (ti_gate_pair)
+    int act = 0;                // 4 or 5: every value of an ungated product passes ti_pointwise_bf16
 };
 
 template <int M, int R, int WPR, int GATED, typename OutT>
@@ -268,10 +270,10 @@ int launch(const Args& a, bool late_start) {
     TI_REQUIRE(blocks <= 0x7FFFFFFFll, "linear (few tokens): %d rows of weights are too many", a.N);
     if (late_start)
         TI_CUDA(ti_launch_after(gemv_kernel<M, R, U, WPR, GATED, OutT>, dim3((unsigned)blocks), dim3(WARPS * 32), 0, a.stream, a.x, a.w,
-                                (OutT*)a.out, a.N, a.K, a.ldx, a.ldw, a.ldo, a.gate_limit));
+                                (OutT*)a.out, a.N, a.K, a.ldx, a.ldw, a.ldo, a.gate_limit, a.act));
     else
         TI_CUDA(ti_launch(gemv_kernel<M, R, U, WPR, GATED, OutT>, dim3((unsigned)blocks), dim3(WARPS * 32), 0, a.stream, a.x, a.w,
-                          (OutT*)a.out, a.N, a.K, a.ldx, a.ldw, a.ldo, a.gate_limit));
+                          (OutT*)a.out, a.N, a.K, a.ldx, a.ldw, a.ldo, a.gate_limit, a.act));
     TI_CHECK_LAUNCH("linear (few tokens)");
     return 0;
 }
@@ -354,8 +356,8 @@ int launch_normed_r(const NormedArgs& a, int rows, int wpr) {
 
 // x[M, K] (row stride ldx), w[N, K] (row stride ldw), both bfloat16, M 1 or 2; out[M, N]
 // bfloat16 or float32.  With `gated`, w's rows are (gate_0, up_0, gate_1, up_1, ...) and out is
-// [M, N / 2] = up * gate / (1 + exp(-gate)) in bfloat16.  K and the strides are multiples of 8
-// elements and the operands 16-byte aligned.  `sms`: the device's multiprocessors; the rows
+// [M, N / 2] = up * gate / (1 + exp(-gate)) in bfloat16 (codes 2 to 5 as for ti_linear_tc).  K and the strides are
+// multiples of 8 elements and the operands 16-byte aligned.  `sms`: the device's multiprocessors; the rows
 // per warp and the warps per row are chosen so that about 32 warps per SM have work.
 extern "C" int ti_linear_gemv(const void* x, const void* w, void* out, int M, int N, int K, long long ldx,
                               long long ldw, long long ldo, int out_f32, int gated, float gate_limit, int sms, int late_start,
@@ -365,11 +367,13 @@ extern "C" int ti_linear_gemv(const void* x, const void* w, void* out, int M, in
     TI_REQUIRE(K % 8 == 0 && ldx % 8 == 0 && ldw % 8 == 0, "linear (few tokens): K and the row strides must be multiples of 8 elements");
     TI_REQUIRE((reinterpret_cast<uintptr_t>(x) & 15) == 0 && (reinterpret_cast<uintptr_t>(w) & 15) == 0,
                "linear (few tokens): operands must be 16-byte aligned");
-    TI_REQUIRE(!gated || (N % 2 == 0 && !out_f32), "linear (few tokens): a gated product needs an even number of weight rows and a bfloat16 result");
+    TI_REQUIRE(gated >= 0 && gated <= 5, "linear (few tokens): unknown activation %d", gated);
+    TI_REQUIRE(!gated || ((gated >= 4 || N % 2 == 0) && !out_f32), "linear (few tokens): a gated product needs an even number of weight rows and a bfloat16 result");
     int rows, wpr;
     choose_shape(M, N, K, sms, &rows, &wpr);
     Args a{(const bf16*)x, (const bf16*)w, out, N, K, ldx, ldw, ldo, stream};
     a.gate_limit = gate_limit;
+    if (gated >= 4) { a.act = gated; gated = 0; }
     return M == 1 ? launch_m<1>(a, out_f32, gated, rows, wpr, late_start != 0) : launch_m<2>(a, out_f32, gated, rows, wpr, late_start != 0);
 }
 

@@ -398,14 +398,7 @@ __global__ void moe_act_pair_vec_kernel(const bf16* __restrict__ gu, bf16* __res
     }
 }
 
-// An ungated activation.  KIND 0: the squared ReLU; 1: gelu by the error function, z (1 + erf(z / sqrt(2))) / 2.
-template <int KIND>
-__device__ __forceinline__ float pointwise_act(float z) {
-    if constexpr (KIND == 0) { const float v = fmaxf(z, 0.f); return v * v; }
-    else return 0.5f * z * (1.0f + erff(z * 0.70710678118654752f));
-}
-
-// the same over 16-byte pieces of bfloat16
+// an ungated activation (ti_pointwise) over 16-byte pieces of bfloat16
 template <int KIND>
 __global__ void pointwise_act_vec_kernel(const bf16* __restrict__ x, bf16* __restrict__ out, long long n8) {
     ti_pdl_trigger();
@@ -418,7 +411,7 @@ __global__ void pointwise_act_vec_kernel(const bf16* __restrict__ x, bf16* __res
         bf16* op = reinterpret_cast<bf16*>(&o4);
 #pragma unroll
         for (int e = 0; e < 8; e++) {
-            op[e] = from_f32<bf16>(pointwise_act<KIND>(to_f32(vp[e])));
+            op[e] = from_f32<bf16>(ti_pointwise_bf16(to_f32(vp[e]), KIND));
         }
         reinterpret_cast<uint4*>(out)[i] = o4;
     }
@@ -463,7 +456,7 @@ __global__ void pointwise_act_kernel(const T* __restrict__ x, T* __restrict__ ou
     ti_pdl_sync();
     x = ti_dependent(x);
     for (long long i = blockIdx.x * (long long)blockDim.x + threadIdx.x; i < n; i += (long long)gridDim.x * blockDim.x)
-        out[i] = from_f32<T>(pointwise_act<KIND>(to_f32(x[i])));
+        out[i] = from_f32<T>(sizeof(T) == 2 ? ti_pointwise_bf16(to_f32(x[i]), KIND) : ti_pointwise(to_f32(x[i]), KIND));
 }
 
 }  // namespace
@@ -595,13 +588,13 @@ extern "C" int ti_moe_combine_indexed(const void* z, const int* pad_of_pair, voi
     });
 }
 
-// out[i] = act(x[i]) in 32-bit with one rounding; kind 0: squared ReLU, 1: gelu (error function).
+// out[i] = act(x[i]) in 32-bit with one rounding; kind 4: squared ReLU, 5: gelu (see ti_pointwise).
 extern "C" int ti_pointwise_act(const void* x, void* out, long long n, int kind, int dtype, cudaStream_t stream) {
     if (n == 0) return 0;
-    TI_REQUIRE(n > 0 && (kind == 0 || kind == 1), "pointwise_act: bad size or unknown activation %d", kind);
+    TI_REQUIRE(n > 0 && (kind == 4 || kind == 5), "pointwise_act: bad size or unknown activation %d", kind);
     if (dtype == TI_BF16 && n % 8 == 0 && (((uintptr_t)x | (uintptr_t)out) & 15) == 0) {
         const long long n8 = n / 8, want = (n8 + 255) / 256;
-        auto kernel = kind == 0 ? pointwise_act_vec_kernel<0> : pointwise_act_vec_kernel<1>;
+        auto kernel = kind == 4 ? pointwise_act_vec_kernel<4> : pointwise_act_vec_kernel<5>;
         TI_CUDA(ti_launch_class<1>(kernel, dim3((unsigned)(want < 148 * 16 ? want : 148 * 16)), dim3(256), 0, stream, (const bf16*)x, (bf16*)out,
                                    n8));
         TI_CHECK_LAUNCH("pointwise_act");
@@ -612,7 +605,7 @@ extern "C" int ti_pointwise_act(const void* x, void* out, long long n, int kind,
         const int threads = 256;
         const long long want = (n + threads - 1) / threads;
         const int blocks = (int)(want < 148 * 16 ? want : 148 * 16);
-        auto kernel = kind == 0 ? pointwise_act_kernel<T, 0> : pointwise_act_kernel<T, 1>;
+        auto kernel = kind == 4 ? pointwise_act_kernel<T, 4> : pointwise_act_kernel<T, 5>;
         TI_CUDA(ti_launch_class<1>(kernel, dim3(blocks), dim3(threads), 0, stream, (const T*)x, (T*)out, n));
         TI_CHECK_LAUNCH("pointwise_act");
         return 0;

@@ -325,6 +325,27 @@ def linear_swiglu(x: torch.Tensor, w_pairs: torch.Tensor, act: str = "silu", lim
     return swiglu(linear(x, w_pairs), pairs=True) if act == "silu" else gated_act(linear(x, w_pairs), act, pairs=True, limit=limit)
 
 
+def linear_act(x: torch.Tensor, w: torch.Tensor, act: str) -> torch.Tensor:
+    """act(x[M, K] times w[N, K] transposed) -> [M, N] with an activation that works value by value (``POINTWISE_ACTS``):
+    in the product's epilogue, on its 32-bit results, where the tensor-core kernels take the shape, else by a kernel of
+    its own."""
+    if act not in POINTWISE_ACTS:
+        raise KernelError(f"linear_act: unknown activation {act!r}; known: {sorted(POINTWISE_ACTS)}")
+    _need_cuda(x, w, what="linear_act")
+    if x.dim() != 2 or w.dim() != 2 or x.shape[1] != w.shape[1] or x.dtype != w.dtype:
+        raise KernelError(f"linear_act: {tuple(x.shape)} {x.dtype} and {tuple(w.shape)} {w.dtype} do not contract")
+    from . import gemm
+    M, K = x.shape
+    N = w.shape[0]
+    ldx, ldw = _row_stride(x, "linear x"), _row_stride(w, "linear w")
+    if gemm.tc_eligible(x, w, K, ldx, ldw):
+        out = torch.empty((M, N), dtype=x.dtype, device=x.device)
+        gemm.run(x, w, out, M, N, K, ldx, ldw, gated=POINTWISE_ACTS[act])
+        return out
+    from .moe import pointwise_act
+    return pointwise_act(linear(x, w), act)
+
+
 def qk_norm_rope_store(q, k, v, q_w, k_w, eps, tables, batch, mem) -> None:
     """In place on the views q[M, heads, d], k[M, kv_heads, d]: per-head RMS norm (when a
     weight is given), rotation by the cos/sin ``tables`` (when given), and the store of k and
@@ -544,6 +565,7 @@ def testing_wait_runs_out(limit: int = 10000) -> bool:
 
 
 GATE_ACTS = {"silu": 0, "gelu_tanh": 1, "clamped_swish": 2}
+POINTWISE_ACTS = {"relu2": 4, "gelu": 5}      # activations without a gate; the products' codes (csrc/common.cuh: ti_pointwise)
 
 
 def gated_act(gu: torch.Tensor, act: str, pairs: bool = False, limit: float = 0.0) -> torch.Tensor:

@@ -79,7 +79,7 @@ def tc_eligible(x, w, K, ldx, ldw) -> bool:
 def run(x, w, out, M, N, K, ldx, ldw, gated: int = 0, late_start: bool = False, gate_limit: float = 0.0) -> None:
     """``gated``: 1 (or True) for up * silu(gate), 2 for up * gelu(gate) in the tanh form, 3 for the clamped pair
     g' sigmoid(1.702 g') (u' + 1) with g' = min(gate, gate_limit), u' = clamp(up, -gate_limit, gate_limit), over paired
-    weight rows; only for shapes the tensor-core kernel takes (see tc_eligible).  ``late_start``: the
+    weight rows; 4 and 5: no pairs, every value through the squared ReLU or gelu; only for shapes the tensor-core kernel takes (see tc_eligible).  ``late_start``: the
     few-token kernels start only when the kernel before them has finished (csrc/gemm_skinny.cu)."""
     lib = library()
     out_f32 = 1 if (out.dtype == torch.float32 and x.dtype != torch.float32) else 0

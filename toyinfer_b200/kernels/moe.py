@@ -6,17 +6,15 @@ from ctypes import c_float, c_int, c_longlong, c_void_p
 
 import torch
 
-from . import KernelError, _call, _code, _i32, _need_cuda, _ptr, _stream
+from . import POINTWISE_ACTS, KernelError, _call, _code, _i32, _need_cuda, _ptr, _stream
 from .wide import _fn
 
 P, I, L, F = c_void_p, c_int, c_longlong, c_float
 
 
-POINTWISE_ACTS = {"relu2": 0, "gelu": 1}
-
-
 def pointwise_act(x: torch.Tensor, act: str) -> torch.Tensor:
-    """An ungated activation, elementwise in 32-bit with one rounding: "relu2" max(x, 0)^2, "gelu" x (1 + erf(x / sqrt(2))) / 2."""
+    """An ungated activation, elementwise in 32-bit with one rounding: "relu2" max(x, 0)^2, "gelu" x (1 + erf(x / sqrt(2))) / 2
+    (bfloat16: by a published approximation that is far below its rounding)."""
     _need_cuda(x, what="pointwise_act")
     if act not in POINTWISE_ACTS:
         raise KernelError(f"pointwise_act: unknown activation {act!r}; known: {sorted(POINTWISE_ACTS)}")

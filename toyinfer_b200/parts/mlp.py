@@ -93,14 +93,14 @@ class GatedDense(FeedForward):
 
 
 class UngatedDense(FeedForward):
-    """y = Wdown act(Wup x) with ``act`` "relu2" (the squared ReLU) or "gelu" (by the error function); no gate, no bias."""
+    """y = Wdown act(Wup x) with ``act`` "relu2" (the squared ReLU) or "gelu" (by the error function); no gate, no bias.  The activation runs in
+    the up product's epilogue on the tensor-core kernels (kernels.linear_act)."""
 
     captures_start = True
 
     def __init__(self, ctx: BuildContext, prefix: str, intermediate_size: int, act: str = "relu2", names: Optional[Dict[str, str]] = None):
-        from ..kernels.moe import POINTWISE_ACTS
-        if act not in POINTWISE_ACTS:
-            raise ValueError(f"feed-forward at {prefix!r}: unknown activation {act!r}; known: {sorted(POINTWISE_ACTS)}")
+        if act not in K.POINTWISE_ACTS:
+            raise ValueError(f"feed-forward at {prefix!r}: unknown activation {act!r}; known: {sorted(K.POINTWISE_ACTS)}")
         self.hidden = ctx.hidden_size
         self.act = act
         self.inter = int(intermediate_size)
@@ -118,8 +118,7 @@ class UngatedDense(FeedForward):
         self.w_down = tensors.pop(self.names["down"]).contiguous()
 
     def forward(self, x, batch) -> torch.Tensor:
-        from ..kernels import moe as KM
-        return K.linear(KM.pointwise_act(K.linear(x, self.w_up), self.act), self.w_down)
+        return K.linear(K.linear_act(x, self.w_up, self.act), self.w_down)
 
 
 class TableMoE(FeedForward):
