@@ -66,9 +66,13 @@ __device__ __forceinline__ void store_chunk(const GemmArgs& g, int i, int b0, in
             }
         }
     } else if (i < g.rows_a) {
-        if (g.gated) {
+        // (one branch for sixteen values: their chains then run side by side)
+        if (g.gated == 4) {
 #pragma unroll
-            for (int e = 0; e < 16; e++) r[e] = ti_pointwise_bf16(r[e], g.gated);
+            for (int e = 0; e < 16; e++) r[e] = ti_pointwise_bf16(r[e], 4);
+        } else if (g.gated == 5) {
+#pragma unroll
+            for (int e = 0; e < 16; e++) r[e] = ti_pointwise_bf16(r[e], 5);
         }
         if (g.transposed) {
             // out[j, i]: the warp's lanes are consecutive i, so each j is one coalesced store
