@@ -255,12 +255,12 @@ def linear(x: torch.Tensor, w: torch.Tensor, out_dtype: Optional[torch.dtype] = 
     return out
 
 
-def linear_bias(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor]) -> torch.Tensor:
+def linear_bias(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor], late_start: bool = False) -> torch.Tensor:
     """x[M, K] times w[N, K] transposed plus bias (float32 [N]) -> [M, N] in x's type: the product's 32-bit result takes
-    the bias before it is rounded.  Without a bias this is ``linear``."""
+    the bias before it is rounded.  Without a bias this is ``linear``; ``late_start`` as there."""
     if bias is None:
-        return linear(x, w)
-    y = linear(x, w, out_dtype=torch.float32)
+        return linear(x, w, late_start=late_start)
+    y = linear(x, w, out_dtype=torch.float32, late_start=late_start)
     M, N = y.shape
     if bias.dtype != torch.float32 or bias.shape != (N,) or not bias.is_contiguous() or not bias.is_cuda:
         raise KernelError(f"linear_bias: the bias must be dense float32 [{N}] on the device")

@@ -142,7 +142,8 @@ class LatentAttention(Mixer):
                 if not store_first:
                     KL.store(lat, batch, mem)
         with ranged(batch, "mixer.out"):
-            return K.linear(a, self.w_o_padded if D else self.w_o)
+            # (single tokens: the attention's blocks have large shared memory; see kernels.linear)
+            return K.linear(a, self.w_o_padded if D else self.w_o, late_start=batch.mode == "extend")
 
 
 register_part("mixer", "latent_attention", LatentAttention)

@@ -120,7 +120,8 @@ class SideBySide(Mixer):
                 L.mix(y[:, :L.n_in], batch, mem[0], out=a[:, :L.n_out], out_scale=self.scales[0])
                 R.mix(y_right, batch, mem[1], out=a[:, L.n_out:], out_scale=self.scales[1])
         with ranged(batch, "mixer.out"):
-            return K.linear_bias(a, self.w_out, self.b_out)
+            # (late: an attention with large shared memory may stand before it)
+            return K.linear_bias(a, self.w_out, self.b_out, late_start=batch.mode == "extend")
 
 
 register_part("mixer", "side_by_side", SideBySide)

@@ -31,6 +31,8 @@ columns of a wider buffer, and its projections' rows handed out, so that it can 
 
 Keys and values of all positions live in the cache; a step first stores its own, then attends over the pages,
 whatever mix of new and cached tokens it brings.  Only the last ``window`` positions are ever read.
+
+The output product of a step of single tokens starts late (kernels.linear): the attention before it has large shared memory.
 """
 from __future__ import annotations
 
@@ -141,7 +143,7 @@ class SigmoidAttention(_WindowAttention):
                           r1=self.r1, r2=self.r2, pb=self.pb, k=qkv[:, H * d:(H + G) * d], v=qkv[:, (H + G) * d:(H + G) * d + G * vd],
                           table=self.table)
         with ranged(batch, "mixer.out"):
-            return K.linear(a, self.w_o)
+            return K.linear(a, self.w_o, late_start=batch.mode == "extend")
 
 
 class DiffAttention(_WindowAttention):
@@ -202,7 +204,7 @@ class DiffAttention(_WindowAttention):
                           k=qkvg[:, nq:nq + G * 2 * d], v=qkvg[:, nq + G * 2 * d:nq + nkv])
             o = KW.diff_combine(a, qkvg[:, nq + nkv:nq + nkv + H] if self.gate else None, H, vd, self.lam, self.diff, self.eps, qkvg.dtype)
         with ranged(batch, "mixer.out"):
-            return K.linear(o, self.w_o)
+            return K.linear(o, self.w_o, late_start=batch.mode == "extend")
 
 
 class KeptWindowAttention(_WindowAttention):
@@ -297,7 +299,7 @@ class KeptWindowAttention(_WindowAttention):
         with ranged(batch, "mixer.attention"):
             a = self.mix(qkv, batch, mem)
         with ranged(batch, "mixer.out"):
-            return K.linear_bias(a, self.w_o, self.b_o)
+            return K.linear_bias(a, self.w_o, self.b_o, late_start=batch.mode == "extend")
 
 
 register_part("mixer", "sigmoid_attention", SigmoidAttention)
