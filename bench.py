@@ -546,8 +546,8 @@ def _mikipel_config(width, heads, layers, kind, vocab=32000):
     else:
         layer = {"type": "delta", "mixer": {"heads": heads, "kv_heads": heads, "dim": 128, "vdim": 128, "conv": 4},
                  "mlp": {"kind": "moe", "expert": {"ff": width}, "router": {"experts": 16, "top": 2}}}
-    return {"architecture": "Mikipel", "vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "embedding": {"scale": 1.0}, "residual_mult": 0.7,
-            "logit_softcap": 30.0, "layers": [json.loads(json.dumps(layer)) for _ in range(layers)], "max_positions": 8192}
+    return {"architecture": "Mikipel", "vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "embedding": {"scale": 1.0}, "residual_mult": 0.6,
+            "logit_softcap": 25.0, "layers": [json.loads(json.dumps(layer)) for _ in range(layers)], "max_positions": 8192}
 
 
 def _qwen3_like(width, heads, layers, vocab=32000):

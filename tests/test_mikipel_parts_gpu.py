@@ -154,7 +154,7 @@ def test_layers_with_shift_and_average_every_way_of_feeding(dtype, ff):
     try:
         blocks = [build_part("block", PartSpec("averaged_parallel", {
             "norm": PartSpec("depth_rmsnorm", {"size": hidden, "eps": eps, "name": "norm1"}), "mixer": PartSpec("doubler_for_a_test"),
-            "feed_forward": PartSpec("ungated_dense", {"intermediate_size": 20, "act": "gelu"}) if ff else None, "depth": i, "mult": 0.7}),
+            "feed_forward": PartSpec("ungated_dense", {"intermediate_size": 20, "act": "gelu"}) if ff else None, "depth": i, "mult": 0.65}),
             ctx_for(dtype, hidden), f"l{i}.") for i in range(3)]
     finally:
         unregister_part("mixer", "doubler_for_a_test")
@@ -171,7 +171,7 @@ def test_layers_with_shift_and_average_every_way_of_feeding(dtype, ff):
             out = 2 * plain.token_shift(z, w[f"l{i}.shift"])
             if ff:
                 out = out + plain.dense_ff(z, {k: w[f"l{i}.mlp.{k}"].double() for k in ("up", "down")})
-            results.append(y + 0.7 * out)
+            results.append(y + 0.65 * out)
             y = plain.depth_average(results, w[f"l{i}.dwa"])
         return y
     xs = inputs([150, 70, 2, 1], hidden, 3, dtype)
