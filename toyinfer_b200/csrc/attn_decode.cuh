@@ -28,6 +28,8 @@ struct DecodeArgs {
     // keep_first: a sequence's first so many positions stay visible behind the window (0: none); out_scale multiplies the
     //           results (where the kernel writes them itself; a merge of splits takes the factor as its own argument).
     int keep_first = 0; float out_scale = 1.f;
+    // gate:     bfloat16 logits [B, heads * hd] (row stride gate_stride) or null: results times sigmoid(gate), on the same terms.
+    const void* gate = nullptr; long long gate_stride = 0;
 };
 
 // One block per (sequence, head); threads over the head's elements.  A split that saw no

@@ -456,7 +456,8 @@ attn_decode_mma_kernel(const __grid_constant__ CUtensorMap k_map, const __grid_c
             fin_o[idx] = acc;
             if (d == 0) { fin_ml[r * 2] = m; fin_ml[r * 2 + 1] = l; }
         } else if (a.n_splits == 1) {
-            const float res = (sig ? acc : (l > 0.f ? acc / l : 0.f)) * (WIN ? a.out_scale : 1.f);
+            float res = (sig ? acc : (l > 0.f ? acc / l : 0.f)) * (WIN ? a.out_scale : 1.f);
+            if (WIN && a.gate) res /= 1.f + expf(-to_f32(ti_dependent((const bf16*)a.gate)[(size_t)b * a.gate_stride + (size_t)h * HD + d]));
             if (WIN && a.out_f32) ((float*)a.out)[(size_t)b * a.o_stride + (size_t)h * HD + d] = res;
             else ((bf16*)a.out)[(size_t)b * a.o_stride + (size_t)h * HD + d] = __float2bfloat16_rn(res);
         } else {
@@ -677,15 +678,17 @@ int launch_win(const tiattn::DecodeArgs& a, int n_seq, cudaStream_t stream) {
 // is read instead when given), else a softmax per map.  q: [B, heads * maps, width / maps]; out: [B, heads * maps, width], bfloat16 or (out_f32)
 // float32, written here when n_splits == 1; else every split leaves part_o [B, heads * maps, splits, width] and part_ml
 // [B, heads * maps, splits, 2] (maximum and sum; both 0 under sigmoid) for the caller's merge.  bfloat16, pages of 64.
-// keep_first: a sequence's first so many positions stay visible behind the window; out_scale multiplies results that are
-// written here (one split).
+// keep_first: a sequence's first so many positions stay visible behind the window; out_scale and sigmoid(gate) (gate:
+// bfloat16 logits [B, heads * maps * width], row stride gate_stride, or null) multiply results that are written here (one
+// split).
 extern "C" int ti_attn_decode_mma_scored(const void* q, long long q_stride, const void* k_pages, const void* v_pages,
                                          const int* page_table, int table_width, int page_size, int ring_rows, int n_pages,
                                          const int* seq_slot, const int* seq_len, int n_seq, int n_heads, int n_kv_heads,
                                          int maps, int width, float scale, int window, int sigmoid, const float* r1,
                                          const float* r2, const float* pb, const float* table, int far, int keep_first,
                                          float out_scale, int n_splits, void* out, long long o_stride,
-                                         int out_f32, float* part_o, float* part_ml, int dtype, cudaStream_t stream) {
+                                         int out_f32, float* part_o, float* part_ml, const void* gate, long long gate_stride,
+                                         int dtype, cudaStream_t stream) {
     if (n_seq == 0) return 0;
     TI_REQUIRE(dtype == TI_BF16, "attention_decode (score rules): bfloat16 only");
     TI_REQUIRE(width == 64 || width == 128, "attention_decode (score rules): rows of %d elements are not 64 or 128", width);
@@ -709,6 +712,7 @@ extern "C" int ti_attn_decode_mma_scored(const void* q, long long q_stride, cons
     a.table = sigmoid ? table : nullptr; a.far = far;
     TI_REQUIRE(keep_first >= 0, "attention_decode (score rules): %d kept first positions", keep_first);
     a.keep_first = window > 0 ? keep_first : 0; a.out_scale = out_scale;
+    a.gate = gate; a.gate_stride = gate_stride;
     return width == 64 ? launch_win<64>(a, n_seq, stream) : launch_win<128>(a, n_seq, stream);
 }
 

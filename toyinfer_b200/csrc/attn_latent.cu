@@ -25,7 +25,7 @@
 //   latent_attn    the attention; a sequence's new tokens follow `seq_start[b]` positions in
 //                  the cache (rows below the start are read from pages, the others from the
 //                  step buffer), any mix of starts and counts in one launch.
-//   latent_expand  o[m, h] = Wuv_h ol[m, h].
+//   latent_expand  o[m, h] = Wuv_h ol[m, h], times sigmoid(gate[m, h]) where a design gates its heads.
 #include "common.cuh"
 #include "attn_decode.cuh"
 
@@ -36,6 +36,12 @@ struct LatentPages {
     const int* page_table; int table_width; int page_size; int ring_rows; int n_pages;
     const int* seq_len;          // each sequence's length after the step (for stores into a ring)
 };
+
+// sigmoid of a head's gate logit: logits [M, heads], row stride in elements
+template <typename T>
+__device__ __forceinline__ float head_gate(const T* gate, long long stride, size_t token, int head) {
+    return 1.0f / (1.0f + expf(-to_f32(gate[token * stride + head])));
+}
 
 template <typename T>
 __device__ __forceinline__ void store_row_to_pages(const LatentPages& kv, int slot, int seq, int pos, int W, const T* row_vals,
@@ -176,7 +182,8 @@ latent_prep_absorb_kernel(const T* __restrict__ d, long long d_stride, const T* 
 template <typename T>
 __global__ void __launch_bounds__(128)
 latent_merge_expand_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml, const T* __restrict__ uv,
-                           T* __restrict__ o, long long o_stride, int n_heads, int vdim, int rank, int n_splits) {
+                           T* __restrict__ o, long long o_stride, int n_heads, int vdim, int rank, int n_splits,
+                           const T* __restrict__ gate, long long gate_stride) {
     ti_pdl_trigger();
     extern __shared__ float res[];       // [rank], then [64] weights
     float* w_s = res + rank;
@@ -194,7 +201,8 @@ latent_merge_expand_kernel(const float* __restrict__ part_o, const float* __rest
         l += w > 0.f ? w * part_ml[(base + s) * 2 + 1] : 0.f;
     }
     __syncthreads();
-    const float inv = l > 0.f ? 1.f / l : 0.f;
+    float inv = l > 0.f ? 1.f / l : 0.f;
+    if (gate) inv *= head_gate(ti_dependent(gate), gate_stride, b, h);      // (the way out is linear)
     for (int e = t; e < rank; e += 128) {
         float acc = 0.f;
         for (int s = 0; s < n_splits; s++) {
@@ -321,11 +329,11 @@ constexpr int EXP_TM = 8, EXP_THREADS = 128, EXP_VB = 16;      // a block: 8 tok
 template <typename T>
 __global__ void __launch_bounds__(EXP_THREADS)
 latent_expand_kernel(const float* __restrict__ ol, const T* __restrict__ uv, T* __restrict__ o, long long o_stride,
-                     int M, int n_heads, int vdim, int rank) {
+                     int M, int n_heads, int vdim, int rank, const T* __restrict__ gate, long long gate_stride) {
     ti_pdl_trigger();
     extern __shared__ float os[];        // [TM][rank]
     ti_pdl_sync();
-    ol = ti_dependent(ol);
+    ol = ti_dependent(ol); gate = ti_dependent(gate);
     const int m0 = blockIdx.x * EXP_TM, h = blockIdx.y, t = threadIdx.x;
     for (int idx = t; idx < EXP_TM * rank; idx += EXP_THREADS) {
         const int mm = idx / rank, r = idx - mm * rank;
@@ -347,7 +355,8 @@ latent_expand_kernel(const float* __restrict__ ol, const T* __restrict__ uv, T* 
 #pragma unroll
         for (int mm = 0; mm < EXP_TM; mm++) {
             const float s = warp_sum(acc[mm]);
-            if (lane == 0 && m0 + mm < M) o[(size_t)(m0 + mm) * o_stride + (size_t)h * vdim + v] = from_f32<T>(s);
+            if (lane == 0 && m0 + mm < M)
+                o[(size_t)(m0 + mm) * o_stride + (size_t)h * vdim + v] = from_f32<T>(gate ? s * head_gate(gate, gate_stride, m0 + mm, h) : s);
         }
     }
 }
@@ -732,7 +741,8 @@ template <int MT, int NTW>
 int launch_decode_mma(const float* qa, const void* lat, float* ol, const int* cu_new, const int* seq_start, const int* seq_slot,
                       int n_seq, int n_heads, int rank, int rot, float scale, int window, const float* sink,
                       const LatentPages& kv, int n_splits, float* part_o, float* part_ml, int n_tok, cudaStream_t stream,
-                      const void* uv = nullptr, void* o = nullptr, long long o_stride = 0, int vdim = 0) {
+                      const void* uv = nullptr, void* o = nullptr, long long o_stride = 0, int vdim = 0, const void* gate = nullptr,
+                      long long gate_stride = 0) {
     constexpr int ROWS = 16 * MT;
     const int W = rank + rot, LD = W + 8;
     const size_t smem = (size_t)(ROWS + DK) * LD * 2 + (size_t)ROWS * (DK + 8) * 2 + ((size_t)ROWS * (DK + 1) + 3 * ROWS) * 4;
@@ -748,7 +758,8 @@ int launch_decode_mma(const float* qa, const void* lat, float* ol, const int* cu
     if (uv) {
         const size_t sm2 = (size_t)(rank + 64) * sizeof(float);
         TI_CUDA(ti_launch_class<4>(latent_merge_expand_kernel<bf16>, dim3(n_tok, n_heads), dim3(128), sm2, stream, (const float*)part_o,
-                                   (const float*)part_ml, (const bf16*)uv, (bf16*)o, o_stride, n_heads, vdim, rank, n_splits));
+                                   (const float*)part_ml, (const bf16*)uv, (bf16*)o, o_stride, n_heads, vdim, rank, n_splits,
+                                   (const bf16*)gate, gate_stride));
         TI_CHECK_LAUNCH("latent_merge_expand");
         return 0;
     }
@@ -864,12 +875,13 @@ extern "C" int ti_latent_prep_absorb(const void* d, long long d_stride, const vo
 extern "C" int ti_latent_decode_takes(int rank, int rot) { return (rank + rot) % 16 == 0 && rank % 8 == 0 && rank <= 512; }
 
 // One query per sequence, bfloat16, tensor cores; the key splits' merge and the way out through uv[heads * vdim, rank] in
-// the second launch: o[n_seq, heads * vdim].  part_o: float32 [n_seq, heads, n_splits, rank], part_ml: [n_seq, heads, n_splits, 2].
+// the second launch: o[n_seq, heads * vdim], head h times sigmoid(gate[., h]) where gate ([n_seq, heads], row stride
+// gate_stride) is given.  part_o: float32 [n_seq, heads, n_splits, rank], part_ml: [n_seq, heads, n_splits, 2].
 extern "C" int ti_latent_decode(const float* qa, const void* lat, const int* cu_new, const int* seq_start, const int* seq_slot,
                                 int n_seq, int n_heads, int rank, int rot, float scale, int window, const float* sink,
                                 const void* pages, const int* page_table, int table_width, int page_size, int ring_rows, int n_pages,
                                 int n_splits, float* part_o, float* part_ml, const void* uv, void* o, long long o_stride, int vdim,
-                                cudaStream_t stream) {
+                                const void* gate, long long gate_stride, cudaStream_t stream) {
     if (n_seq == 0) return 0;
     TI_REQUIRE(n_seq > 0 && n_seq <= 65535 && n_heads > 0 && vdim > 0 && ti_latent_decode_takes(rank, rot), "latent_decode: sizes not taken");
     TI_REQUIRE(n_splits >= 1 && n_splits <= 64 && part_o && part_ml && uv && o, "latent_decode: bad arguments");
@@ -880,7 +892,7 @@ extern "C" int ti_latent_decode(const float* qa, const void* lat, const int* cu_
     LatentPages kv{const_cast<void*>(pages), page_table, table_width, page_size, ring_rows, n_pages, nullptr};
     const bool two = n_heads > 16;
 #define TI_LATENT_DECODE(MT, NTW) launch_decode_mma<MT, NTW>(qa, lat, nullptr, cu_new, seq_start, seq_slot, n_seq, n_heads, rank, rot, scale, \
-                                                            window, sink, kv, n_splits, part_o, part_ml, n_seq, stream, uv, o, o_stride, vdim)
+                                                            window, sink, kv, n_splits, part_o, part_ml, n_seq, stream, uv, o, o_stride, vdim, gate, gate_stride)
     if (rank <= 128) return two ? TI_LATENT_DECODE(2, 4) : TI_LATENT_DECODE(1, 4);
     if (rank <= 256) return two ? TI_LATENT_DECODE(2, 8) : TI_LATENT_DECODE(1, 8);
     return two ? TI_LATENT_DECODE(2, 16) : TI_LATENT_DECODE(1, 16);
@@ -918,7 +930,7 @@ extern "C" int ti_latent_absorb(const void* q, long long q_stride, const void* u
 }
 
 extern "C" int ti_latent_expand(const float* ol, const void* uv, void* o, long long o_stride, int M, int n_heads, int vdim,
-                                int rank, int dtype, cudaStream_t stream) {
+                                int rank, const void* gate, long long gate_stride, int dtype, cudaStream_t stream) {
     if (M == 0) return 0;
     TI_REQUIRE(M > 0 && n_heads > 0 && n_heads <= 65535 && vdim > 0 && rank > 0, "latent_expand: bad sizes");
     const size_t smem = (size_t)EXP_TM * rank * sizeof(float);
@@ -926,7 +938,7 @@ extern "C" int ti_latent_expand(const float* ol, const void* uv, void* o, long l
     return ti_dispatch_dtype(dtype, [&](auto t) -> int {
         using T = decltype(t);
         TI_CUDA(ti_launch(latent_expand_kernel<T>, dim3((M + EXP_TM - 1) / EXP_TM, n_heads, (vdim + EXP_VB - 1) / EXP_VB), dim3(EXP_THREADS), smem, stream, ol,
-                          (const T*)uv, (T*)o, o_stride, M, n_heads, vdim, rank));
+                          (const T*)uv, (T*)o, o_stride, M, n_heads, vdim, rank, (const T*)gate, gate_stride));
         TI_CHECK_LAUNCH("latent_expand");
         return 0;
     });

@@ -66,6 +66,9 @@ struct Args {
     // The first keep_first positions of a sequence stay visible to every later query whatever the window (0: none);
     // results are multiplied by out_scale before they are rounded.
     int keep_first = 0; float out_scale = 1.f;
+    // Results times sigmoid(gate): bfloat16 logits per token, one per result element (gate_heads 0: 16-byte aligned rows) or
+    // one per head; or null.
+    const void* gate = nullptr; long long gate_stride = 0; int gate_heads = 0;
 };
 
 __device__ __forceinline__ float ex2(float x) {
@@ -73,6 +76,8 @@ __device__ __forceinline__ float ex2(float x) {
     asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
     return y;
 }
+
+__device__ __forceinline__ float sigmoid2(float z) { return __fdividef(1.0f, 1.0f + ex2(fminf(-1.4426950408889634f * z, 126.f))); }
 
 // Two floats in one 64-bit register pair, for the packed float32 instructions of sm_100: the
 // softmax warps are bound by how many instructions they issue, and these do two elements each.
@@ -517,13 +522,27 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_c
         if (a.sink != nullptr && m_used > -INFINITY) l_run += ex2(fminf(a.sink[h] * 1.4426950408889634f - m_used, 126.f));
         if (ok) {
             tc_fence_after();
-            const float inv = MODE == 1 ? a.out_scale : l_run > 0.f ? a.out_scale / l_run : 0.f;
+            float inv = MODE == 1 ? a.out_scale : l_run > 0.f ? a.out_scale / l_run : 0.f;
+            const bf16* grow = a.gate && qi < n ? ti_dependent((const bf16*)a.gate) + (size_t)(tok0 + qi) * a.gate_stride : nullptr;
+            if (grow && a.gate_heads) {
+                inv *= sigmoid2(to_f32(grow[h]));
+                grow = nullptr;
+            }
             bf16* orow = (bf16*)a.out + (size_t)(tok0 + qi) * a.o_stride + (size_t)hv * HDV;
             float* orow32 = (float*)a.out + (size_t)(tok0 + qi) * a.o_stride + (size_t)hv * HDV;
 #pragma unroll 1
             for (int c = half * (HDV / 64); c < (half + 1) * (HDV / 64); c++) {
                 float o[32];
                 tmem_ld32(tmem + O_COL + lane_base + c * 32, o);
+                if (grow) {
+#pragma unroll
+                    for (int t4 = 0; t4 < 4; t4++) {
+                        const uint4 g4 = *reinterpret_cast<const uint4*>(grow + (size_t)hv * HDV + c * 32 + t4 * 8);
+                        const bf16* g = reinterpret_cast<const bf16*>(&g4);
+#pragma unroll
+                        for (int e = 0; e < 8; e++) o[t4 * 8 + e] *= sigmoid2(to_f32(g[e]));
+                    }
+                }
                 if (qi < n && a.out_f32) {
 #pragma unroll
                     for (int e = 0; e < 32; e += 4)
@@ -630,11 +649,13 @@ extern "C" int ti_attn_prefill_tc(const void* q, const void* k, const void* v, v
                           : launch<128, false>(qm, km, vm, km, vm, a, n_seq, max_new, stream);
 }
 
-// The same with sinks: float32 sink[n_heads], exp(sink_h) is added to head h's softmax denominator.
+// The same with sinks (float32 sink[n_heads], exp(sink_h) is added to head h's softmax denominator; or null) and a gate per
+// head (bfloat16 logits [n_tokens, n_heads], row stride gate_stride: head h's results times sigmoid(gate_h); or null).
 extern "C" int ti_attn_prefill_tc_sink(const void* q, const void* k, const void* v, void* out,
                                        long long q_stride, long long k_stride, long long v_stride, long long o_stride,
                                        const int* cu_new, int n_seq, int max_new, int n_tokens, int n_heads, int n_kv_heads,
-                                       int head_dim, float scale, int window, const float* sink, cudaStream_t stream) {
+                                       int head_dim, float scale, int window, const float* sink, const void* gate,
+                                       long long gate_stride, cudaStream_t stream) {
     if (n_seq == 0 || max_new == 0) return 0;
     CUtensorMap qm, km, vm;
     if (int rc = check_common("attention_prefill", q, k, v, out, q_stride, k_stride, v_stride, o_stride, n_seq, n_tokens,
@@ -642,6 +663,7 @@ extern "C" int ti_attn_prefill_tc_sink(const void* q, const void* k, const void*
     Args a = {};
     a.cu_new = cu_new; a.n_heads = n_heads; a.n_kv_heads = n_kv_heads; a.scale = scale; a.window = window;
     a.out = out; a.o_stride = o_stride; a.sink = sink;
+    a.gate = gate; a.gate_stride = gate_stride; a.gate_heads = 1;
     return head_dim == 64 ? launch<64, false>(qm, km, vm, km, vm, a, n_seq, max_new, stream)
                           : launch<128, false>(qm, km, vm, km, vm, a, n_seq, max_new, stream);
 }
@@ -734,14 +756,15 @@ extern "C" int ti_attn_chunk_tc(const void* q, const void* k, const void* v, voi
 // o_stride in elements of that type.  seq_start null: every sequence starts at position 0 and the pages are not read.
 // Otherwise k_pages [pages, kv_heads, 64, maps * dim] and v_pages [pages, kv_heads, 64, vdim] hold the positions
 // before the step's.  dist_bias: float32 [heads, far + 1] or null.  window <= 0: every earlier position.  keep_first: a
-// sequence's first so many positions stay visible behind the window; out_scale multiplies the results.
+// sequence's first so many positions stay visible behind the window; out_scale multiplies the results, and so does
+// sigmoid(gate) (gate: bfloat16 logits [n_tokens, heads * maps * vdim], row stride gate_stride, or null).
 extern "C" int ti_attn_window_tc(const void* q, const void* k, const void* v, void* out,
                                  long long q_stride, long long k_stride, long long v_stride, long long o_stride, int out_f32,
                                  const int* cu_new, const int* seq_start, const int* seq_slot, int n_seq, int max_new,
                                  int n_tokens, int n_heads, int n_kv_heads, int maps, int dim, int vdim, float scale, int window,
                                  int mode, const void* k_pages, const void* v_pages, const int* page_table, int table_width,
                                  int page_size, int n_pages, const float* dist_bias, int far, int keep_first, float out_scale,
-                                 cudaStream_t stream) {
+                                 const void* gate, long long gate_stride, cudaStream_t stream) {
     if (n_seq == 0 || max_new == 0) return 0;
     const char* what = "attention_window (tcgen05)";
     TI_REQUIRE(keep_first >= 0, "%s: %d kept first positions", what, keep_first);
@@ -750,6 +773,7 @@ extern "C" int ti_attn_window_tc(const void* q, const void* k, const void* v, vo
     TI_REQUIRE(n_seq <= 65535 && n_tokens <= 65535 * BQ, "%s: too many sequences or tokens for one launch", what);
     TI_REQUIRE(mode == 0 || mode == 1, "%s: unknown mode %d", what, mode);
     TI_REQUIRE(scale > 0.f && (!dist_bias || far >= 0), "%s: needs a positive scale", what);
+    TI_REQUIRE(!gate || ((reinterpret_cast<uintptr_t>(gate) & 15) == 0 && gate_stride % 8 == 0), "%s: the gate's rows must be 16-byte aligned", what);
     TI_REQUIRE(q_stride % 8 == 0 && k_stride % 8 == 0 && v_stride % 8 == 0 && o_stride % (out_f32 ? 4 : 8) == 0,
                "%s: token strides must be multiples of 16 bytes", what);
     TI_REQUIRE(((reinterpret_cast<uintptr_t>(q) | reinterpret_cast<uintptr_t>(k) | reinterpret_cast<uintptr_t>(v) |
@@ -774,6 +798,7 @@ extern "C" int ti_attn_window_tc(const void* q, const void* k, const void* v, vo
     a.seq_start = seq_start; a.seq_slot = seq_slot; a.page_table = page_table; a.table_width = table_width;
     a.ring_rows = 0; a.n_pages = n_pages; a.dist_bias = dist_bias; a.far = far;
     a.keep_first = window > 0 ? keep_first : 0; a.out_scale = out_scale;
+    a.gate = gate; a.gate_stride = gate_stride;
     auto go = [&](auto dk, auto dv) -> int {
         constexpr int DK = decltype(dk)::value, DV = decltype(dv)::value;
         if (mode == 1) return paged ? launch<DK, true, DV, 1>(qm, km, vm, kpm, vpm, a, n_seq, max_new, stream)

@@ -27,6 +27,8 @@
 //   biases, norms every head of q and of k over its own `dim` elements with one weight [dim] for all
 //   heads (each optional), rotates the first `rot` elements of every head of q and k, pairing either
 //   (e, e + rot/2) or neighbours (2e, 2e + 1) with the same tables, writes back and stores k and v.
+//   A query may be multiplied by a temperature that grows with its position, and a value may be
+//   blended with another layer's value of the same token before it is stored (HeadExtras).
 // attn_window: any number of new tokens per sequence after any number of cached ones; all keys
 //   are read from the pages, so the step's own must be stored first.  Grid (query tiles of 32,
 //   virtual heads, sequences), 128 threads: thread t works on query row t / 4; its 4 threads split
@@ -38,6 +40,9 @@
 //   kernel when there are several (ti_attn_window_merge serves the tensor-core decode kernel of
 //   attn_decode_mma.cu the same way, which takes bfloat16 single tokens where it can).
 // diff_combine: o = a1 - lambda a2 of the two maps' outputs, o / rms(o) * (1 - diff) * sigmoid(gate).
+//
+// The attention kernels may multiply every element of their result by sigmoid(gate), the gate's
+// logits in rows beside the queries (Gate), before it is rounded.
 #include "common.cuh"
 
 #include <algorithm>
@@ -51,6 +56,28 @@ struct Pages {
 };
 
 __device__ __forceinline__ float sigmoidf(float x) { return 1.0f / (1.0f + expf(-x)); }
+
+// A logit per element of a token's results (engine type, row stride in elements), or none.
+struct Gate {
+    const void* logits; long long stride;
+};
+
+template <typename T>
+__device__ __forceinline__ float gated(float o, const Gate& g, size_t token, int element) {
+    return g.logits ? o * sigmoidf(to_f32(((const T*)g.logits)[token * g.stride + element])) : o;
+}
+
+// What attn_head_prepare may do beside norms and rotation.  every > 0: the query at position p is multiplied by
+// 1 + coef ln(floor((p + 1) / every) + 1) after its norm.  first: values of the same tokens [M, kv_heads * vdim] (row stride
+// first_stride), v <- (1 - mix) v + mix first after the bias.
+struct HeadExtras {
+    float coef; int every;
+    const void* first; long long first_stride; float mix;
+};
+
+__device__ __forceinline__ float query_temperature(const HeadExtras& x, int p) {
+    return x.every > 0 ? 1.0f + x.coef * logf((float)((p + 1) / x.every + 1)) : 1.0f;
+}
 
 template <typename T>
 __global__ void attn_window_prepare_kernel(T* __restrict__ qkv, long long ld, const float* __restrict__ bias,
@@ -242,7 +269,7 @@ __global__ void attn_head_prepare_kernel(T* __restrict__ qkv, long long ld, cons
                                          const float* __restrict__ cos_t, const float* __restrict__ sin_t, int rot, int pairing,
                                          int max_pos, const int* __restrict__ tok_pos, const int* __restrict__ tok_seq,
                                          const int* __restrict__ seq_slot, Pages pg, long long rows, int H, int G, int dim, int vdim,
-                                         int width) {
+                                         int width, HeadExtras ex) {
     ti_pdl_trigger();
     extern __shared__ float sm[];
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
@@ -263,9 +290,11 @@ __global__ void attn_head_prepare_kernel(T* __restrict__ qkv, long long ld, cons
     ti_pdl_sync();
     qkv = ti_dependent(qkv);
     T* row = qkv + (size_t)m * ld + off;
+    const T* first = ex.first && kind == 2 ? ti_dependent((const T*)ex.first) + (size_t)m * ex.first_stride + head * vdim : nullptr;
     float ss = 0.f;
     for (int i = lane; i < n; i += 32) {
-        const float v = to_f32(row[i]) + (bias ? bias[off + i] : 0.f);
+        float v = to_f32(row[i]) + (bias ? bias[off + i] : 0.f);
+        if (first) v = (1.0f - ex.mix) * v + ex.mix * to_f32(first[i]);
         x[i] = v;
         ss = fmaf(v, v, ss);
     }
@@ -273,6 +302,10 @@ __global__ void attn_head_prepare_kernel(T* __restrict__ qkv, long long ld, cons
     if (w) {
         const float inv = rsqrtf(warp_sum(ss) / (float)n + eps);
         for (int i = lane; i < n; i += 32) x[i] = x[i] * inv * w[i];
+    }
+    if (kind == 0 && ex.every > 0) {
+        const float warm = query_temperature(ex, p);
+        for (int i = lane; i < n; i += 32) x[i] *= warm;
     }
     __syncwarp();
     const int pp = (page >= 0 && page < pg.n_pages) ? page : 0;       // page 0 is scratch
@@ -304,11 +337,12 @@ attn_window_kernel(const T* __restrict__ q, long long q_stride, OT* __restrict__
                    const int* __restrict__ cu_new, const int* __restrict__ seq_start, const int* __restrict__ seq_slot,
                    Pages pg, const float* __restrict__ r1, const float* __restrict__ r2, const float* __restrict__ pb,
                    int n_heads, int n_kv_heads, int maps, int dim, int vdim, float scale, int window, int keep_first,
-                   float out_scale) {
+                   float out_scale, Gate gate) {
     ti_pdl_trigger();
     extern __shared__ float sm[];
     ti_pdl_sync();
     q = ti_dependent(q);
+    gate.logits = ti_dependent((const T*)gate.logits);
     const int ldk = dim + 1, ldv = vdim + 1;
     float* Qs = sm;                      // [BQ][dim + 1]
     float* Ks = Qs + BQ * ldk;           // [BKV][dim + 1]
@@ -429,7 +463,8 @@ attn_window_kernel(const T* __restrict__ q, long long q_stride, OT* __restrict__
         OT* orow = out + (size_t)(tok0 + qi - start) * o_stride + (size_t)hv * vdim;
 #pragma unroll
         for (int c = 0; c < MAXC; c++)
-            if (c < nc && c4 + 4 * c < vdim) orow[c4 + 4 * c] = from_f32<OT>(acc[c] * inv);
+            if (c < nc && c4 + 4 * c < vdim)
+                orow[c4 + 4 * c] = from_f32<OT>(gated<T>(acc[c] * inv, gate, (size_t)(tok0 + qi - start), hv * vdim + c4 + 4 * c));
     }
 }
 
@@ -461,7 +496,8 @@ __global__ void attn_head_prepare_vec_kernel(bf16* __restrict__ qkv, long long l
                                              const float* __restrict__ q_w, const float* __restrict__ k_w, float eps,
                                              const float* __restrict__ cos_t, const float* __restrict__ sin_t, int rot, int pairing,
                                              int max_pos, const int* __restrict__ tok_pos, const int* __restrict__ tok_seq,
-                                             const int* __restrict__ seq_slot, Pages pg, long long rows, int H, int G, int dim, int vdim) {
+                                             const int* __restrict__ seq_slot, Pages pg, long long rows, int H, int G, int dim, int vdim,
+                                             HeadExtras ex) {
     ti_pdl_trigger();
     constexpr int E = 8, RPW = 32 / LANES;
     const int lane = threadIdx.x & 31, l = lane % LANES;
@@ -501,6 +537,12 @@ __global__ void attn_head_prepare_vec_kernel(bf16* __restrict__ qkv, long long l
             const float4 b0 = *reinterpret_cast<const float4*>(bias + off + i0), b1 = *reinterpret_cast<const float4*>(bias + off + i0 + 4);
             x[0] += b0.x; x[1] += b0.y; x[2] += b0.z; x[3] += b0.w; x[4] += b1.x; x[5] += b1.y; x[6] += b1.z; x[7] += b1.w;
         }
+        if (ex.first && kind == 2) {
+            float f[E];
+            load_run<bf16, E>(ti_dependent((const bf16*)ex.first) + (size_t)m * ex.first_stride + head * vdim + i0, f, true);
+#pragma unroll
+            for (int e = 0; e < E; e++) x[e] = (1.0f - ex.mix) * x[e] + ex.mix * f[e];
+        }
 #pragma unroll
         for (int e = 0; e < E; e++) ss = fmaf(x[e], x[e], ss);
     }
@@ -510,6 +552,11 @@ __global__ void attn_head_prepare_vec_kernel(bf16* __restrict__ qkv, long long l
         const float inv = rsqrtf(ss / (float)n + eps);
 #pragma unroll
         for (int e = 0; e < E; e++) x[e] = x[e] * inv * w[i0 + e];
+    }
+    if (kind == 0 && ex.every > 0) {
+        const float warm = query_temperature(ex, p);
+#pragma unroll
+        for (int e = 0; e < E; e++) x[e] *= warm;
     }
     if (cos_t) {                // (the same for the whole grid: every lane takes part in the exchange)
         if (pairing) {
@@ -550,7 +597,7 @@ attn_window_decode_kernel(const T* __restrict__ q, long long q_stride, OT* __res
                           const int* __restrict__ seq_len, const int* __restrict__ seq_slot, Pages pg,
                           const float* __restrict__ r1, const float* __restrict__ r2, const float* __restrict__ pb,
                           int n_heads, int n_kv_heads, int maps, int dim, int vdim, float scale, int window, int keep_first,
-                          float out_scale, int splits, float* __restrict__ part_o, float* __restrict__ part_ml) {
+                          float out_scale, int splits, float* __restrict__ part_o, float* __restrict__ part_ml, Gate gate) {
     ti_pdl_trigger();
     extern __shared__ __align__(16) float dsm[];         // q: [GH][dim]; o: [DEC_WARPS][GH][32 * VPL]; m, l: [DEC_WARPS][GH][2]
     float* q_sh = dsm;
@@ -558,6 +605,7 @@ attn_window_decode_kernel(const T* __restrict__ q, long long q_stride, OT* __res
     float* ml_sh = o_sh + DEC_WARPS * GH * 32 * VPL;
     ti_pdl_sync();
     q = ti_dependent(q);
+    gate.logits = ti_dependent((const T*)gate.logits);
     const int b = blockIdx.z, sp = blockIdx.x;
     const int group = n_heads / n_kv_heads, cpg = group / GH;        // chunks of GH heads per kv head and map
     const int kvh = blockIdx.y / (maps * cpg), rem = blockIdx.y - kvh * maps * cpg;
@@ -693,7 +741,7 @@ attn_window_decode_kernel(const T* __restrict__ q, long long q_stride, OT* __res
             for (int w = 0; w < DEC_WARPS; w++) o = fmaf(o_sh[(w * GH + g) * 32 * VPL + d], f[w], o);
             if (splits == 1) {
                 if constexpr (MODE == 0) o = l_all > 0.f ? o / l_all : 0.f;
-                out[(size_t)b * o_stride + (size_t)hv * vdim + d] = from_f32<OT>(o * out_scale);
+                out[(size_t)b * o_stride + (size_t)hv * vdim + d] = from_f32<OT>(gated<T>(o * out_scale, gate, b, hv * vdim + d));
             } else {
                 part_o[(((size_t)b * n_heads * maps + hv) * splits + sp) * vdim + d] = o;
             }
@@ -705,9 +753,9 @@ attn_window_decode_kernel(const T* __restrict__ q, long long q_stride, OT* __res
     }
 }
 
-template <typename OT, int MODE>
+template <typename T, typename OT, int MODE>
 __global__ void attn_window_merge_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml, OT* __restrict__ out,
-                                         long long o_stride, int n_virtual, int vdim, int splits, float out_scale) {
+                                         long long o_stride, int n_virtual, int vdim, int splits, float out_scale, Gate gate) {
     ti_pdl_trigger();
     ti_pdl_sync();
     part_o = ti_dependent(part_o); part_ml = ti_dependent(part_ml);
@@ -718,7 +766,7 @@ __global__ void attn_window_merge_kernel(const float* __restrict__ part_o, const
         for (int d = threadIdx.x; d < vdim; d += blockDim.x) {
             float o = 0.f;
             for (int s = 0; s < splits; s++) o += po[(size_t)s * vdim + d];
-            out[(size_t)b * o_stride + (size_t)hv * vdim + d] = from_f32<OT>(o * out_scale);
+            out[(size_t)b * o_stride + (size_t)hv * vdim + d] = from_f32<OT>(gated<T>(o * out_scale, gate, b, hv * vdim + d));
         }
         return;
     }
@@ -730,7 +778,8 @@ __global__ void attn_window_merge_kernel(const float* __restrict__ part_o, const
         float o = 0.f;
         for (int s = 0; s < splits; s++)
             if (ml[2 * s] > -INFINITY) o = fmaf(po[(size_t)s * vdim + d], expf(ml[2 * s] - m_all), o);
-        out[(size_t)b * o_stride + (size_t)hv * vdim + d] = from_f32<OT>(l_all > 0.f ? o / l_all * out_scale : 0.f);
+        out[(size_t)b * o_stride + (size_t)hv * vdim + d] =
+            from_f32<OT>(gated<T>(l_all > 0.f ? o / l_all * out_scale : 0.f, gate, b, hv * vdim + d));
     }
 }
 
@@ -817,14 +866,19 @@ extern "C" int ti_attn_window_prepare(void* qkv, long long ld, const float* bias
 
 // qkv: [M, >= heads * dim + kv_heads * (dim + vdim)] of the engine's type, row stride ld (columns after q, k, v are left
 // alone); bias: float32 of q, k and v's length or null; q_w, k_w: float32 [dim] or null (one weight for all heads); cos_t,
-// sin_t: float32 [max_pos, rot / 2] or null; pairing 0: elements (e, e + rot / 2) turn together, 1: (2e, 2e + 1).
+// sin_t: float32 [max_pos, rot / 2] or null; pairing 0: elements (e, e + rot / 2) turn together, 1: (2e, 2e + 1).  temp_every
+// > 0: queries times 1 + temp_coef ln(floor((p + 1) / temp_every) + 1); first: [M, kv_heads * vdim] of the engine's type with
+// row stride first_stride or null: values become (1 - mix) v + mix first.
 extern "C" int ti_attn_head_prepare(void* qkv, long long ld, const float* bias, const float* q_w, const float* k_w, float eps,
                                     const float* cos_t, const float* sin_t, int rot, int pairing, int max_pos, const int* tok_pos,
                                     const int* tok_seq, const int* seq_slot, void* k_pages, void* v_pages, const int* page_table,
                                     int table_width, int page_size, int n_pages, int M, int n_heads, int n_kv_heads, int dim,
-                                    int vdim, int dtype, cudaStream_t stream) {
+                                    int vdim, float temp_coef, int temp_every, const void* first, long long first_stride, float mix,
+                                    int dtype, cudaStream_t stream) {
     if (M == 0) return 0;
-    TI_REQUIRE(M > 0 && n_heads > 0 && n_kv_heads > 0 && dim > 0 && vdim > 0, "attn_head_prepare: bad sizes");
+    TI_REQUIRE(M > 0 && n_heads > 0 && n_kv_heads > 0 && dim > 0 && vdim > 0 && temp_every >= 0, "attn_head_prepare: bad sizes");
+    TI_REQUIRE(!first || first_stride >= (long long)n_kv_heads * vdim, "attn_head_prepare: the values to blend in do not fit the heads");
+    const HeadExtras ex{temp_coef, temp_every, first, first_stride, mix};
     TI_REQUIRE(!cos_t || (sin_t && rot > 0 && rot % 2 == 0 && rot <= dim && max_pos > 0 && (pairing == 0 || pairing == 1)),
                "attn_head_prepare: a rotation of %d of %d elements with tables of %d positions", rot, dim, max_pos);
     if (check_pages("attn_head_prepare", k_pages, v_pages, page_table, table_width, page_size, n_pages)) return 1;
@@ -836,12 +890,13 @@ extern "C" int ti_attn_head_prepare(void* qkv, long long ld, const float* bias, 
     auto lanes = [](int n) { return n == 64 || n == 128 || n == 256; };
     auto a16 = [](const void* q) { return (reinterpret_cast<uintptr_t>(q) & 15) == 0; };
     if (dtype == TI_BF16 && lanes(dim) && lanes(vdim) && ld % 8 == 0 && a16(qkv) && a16(k_pages) && a16(v_pages) && a16(bias) &&
+        a16(first) && first_stride % 8 == 0 &&
         (!cos_t || pairing == 1 || (rot / 2) % 8 == 0)) {
         const int group = std::max(dim, vdim) / 8;          // lanes that stand for a head
         const long long warps = (rows + 32 / group - 1) / (32 / group);
         const dim3 grid((unsigned)((warps + 3) / 4)), block(128);
 #define TI_HEAD_PREPARE(L) TI_CUDA(ti_launch_class<2>(attn_head_prepare_vec_kernel<L>, grid, block, 0, stream, (bf16*)qkv, ld, bias, q_w, k_w, eps, \
-            cos_t, sin_t, cos_t ? rot : 0, pairing, max_pos, tok_pos, tok_seq, seq_slot, pg, rows, n_heads, n_kv_heads, dim, vdim))
+            cos_t, sin_t, cos_t ? rot : 0, pairing, max_pos, tok_pos, tok_seq, seq_slot, pg, rows, n_heads, n_kv_heads, dim, vdim, ex))
         if (group == 8) TI_HEAD_PREPARE(8); else if (group == 16) TI_HEAD_PREPARE(16); else TI_HEAD_PREPARE(32);
 #undef TI_HEAD_PREPARE
         TI_CHECK_LAUNCH("attn_head_prepare (a lane a run)");
@@ -851,20 +906,21 @@ extern "C" int ti_attn_head_prepare(void* qkv, long long ld, const float* bias, 
         using T = decltype(t);
         TI_CUDA(ti_launch_class<2>(attn_head_prepare_kernel<T>, dim3((unsigned)((rows + warps - 1) / warps)), dim3(warps * 32), smem, stream,
                                    (T*)qkv, ld, bias, q_w, k_w, eps, cos_t, sin_t, cos_t ? rot : 0, pairing, max_pos, tok_pos, tok_seq,
-                                   seq_slot, pg, rows, n_heads, n_kv_heads, dim, vdim, width));
+                                   seq_slot, pg, rows, n_heads, n_kv_heads, dim, vdim, width, ex));
         TI_CHECK_LAUNCH("attn_head_prepare");
         return 0;
     });
 }
 
 // q: [M, heads * maps, dim] (row stride q_stride); out: [M, heads * maps, vdim] (row stride o_stride), float32 when
-// out_f32 else the engine's type; r1, r2, pb: float32 [heads] or null; mode 0 softmax, 1 sigmoid; window <= 0: all keys.
+// out_f32 else the engine's type; r1, r2, pb: float32 [heads] or null; mode 0 softmax, 1 sigmoid; window <= 0: all keys;
+// gate: logits [M, heads * maps * vdim] of the engine's type with row stride gate_stride, or null.
 extern "C" int ti_attn_window(const void* q, long long q_stride, void* out, long long o_stride, int out_f32, const int* cu_new,
                               const int* seq_start, const int* seq_slot, int n_seq, int max_new, const void* k_pages,
                               const void* v_pages, const int* page_table, int table_width, int page_size, int n_pages,
                               const float* r1, const float* r2, const float* pb, int n_heads, int n_kv_heads, int maps, int dim,
-                              int vdim, float scale, int window, int keep_first, float out_scale, int mode, int dtype,
-                              cudaStream_t stream) {
+                              int vdim, float scale, int window, int keep_first, float out_scale, int mode, const void* gate,
+                              long long gate_stride, int dtype, cudaStream_t stream) {
     if (n_seq == 0 || max_new == 0) return 0;
     TI_REQUIRE(n_seq > 0 && max_new > 0 && n_heads > 0 && n_kv_heads > 0 && n_heads % n_kv_heads == 0 && maps > 0, "attn_window: bad sizes");
     TI_REQUIRE(dim >= 1 && dim <= 256 && vdim >= 1 && vdim <= 256, "attn_window: heads of %d and %d elements are not supported (up to 256)", dim, vdim);
@@ -888,7 +944,7 @@ extern "C" int ti_attn_window(const void* q, long long q_stride, void* out, long
             }
             TI_CUDA(ti_launch(attn_window_kernel<T, OT, MAXC, MODE>, grid, dim3(THREADS), smem, stream, (const T*)q, q_stride, (OT*)out,
                               o_stride, cu_new, seq_start, seq_slot, pg, r1, r2, pb, n_heads, n_kv_heads, maps, dim, vdim, scale, window,
-                              window > 0 ? keep_first : 0, out_scale));
+                              window > 0 ? keep_first : 0, out_scale, Gate{gate, gate_stride}));
             TI_CHECK_LAUNCH("attn_window");
             return 0;
         };
@@ -911,7 +967,7 @@ extern "C" int ti_attn_window_decode(const void* q, long long q_stride, void* ou
                                      const int* page_table, int table_width, int page_size, int n_pages, const float* r1,
                                      const float* r2, const float* pb, int n_heads, int n_kv_heads, int maps, int dim, int vdim,
                                      float scale, int window, int keep_first, float out_scale, int mode, int splits, float* part_o,
-                                     float* part_ml, int dtype, cudaStream_t stream) {
+                                     float* part_ml, const void* gate, long long gate_stride, int dtype, cudaStream_t stream) {
     if (n_seq == 0) return 0;
     TI_REQUIRE(n_seq > 0 && n_heads > 0 && n_kv_heads > 0 && n_heads % n_kv_heads == 0 && maps > 0 && splits >= 1, "attn_window_decode: bad sizes");
     TI_REQUIRE(dim >= 1 && dim <= 32 * DEC_MAXE && vdim >= 1 && vdim <= 32 * DEC_MAXE,
@@ -941,11 +997,12 @@ extern "C" int ti_attn_window_decode(const void* q, long long q_stride, void* ou
             TI_CUDA(ti_launch_class<3>(attn_window_decode_kernel<T, OT, GH, VPL, MODE>, dim3(splits, n_heads * maps / GH, n_seq),
                                        dim3(DEC_WARPS * 32), smem, stream, (const T*)q, q_stride, (OT*)out, o_stride, seq_len, seq_slot, pg,
                                        r1, r2, pb, n_heads, n_kv_heads, maps, dim, vdim, scale, window, window > 0 ? keep_first : 0, out_scale, splits,
-                                       part_o, part_ml));
+                                       part_o, part_ml, Gate{gate, gate_stride}));
             TI_CHECK_LAUNCH("attn_window_decode");
             if (splits > 1) {
-                TI_CUDA(ti_launch_class<4>(attn_window_merge_kernel<OT, MODE>, dim3(n_heads * maps, n_seq), dim3(64), 0, stream,
-                                           (const float*)part_o, (const float*)part_ml, (OT*)out, o_stride, n_heads * maps, vdim, splits, out_scale));
+                TI_CUDA(ti_launch_class<4>(attn_window_merge_kernel<T, OT, MODE>, dim3(n_heads * maps, n_seq), dim3(64), 0, stream,
+                                           (const float*)part_o, (const float*)part_ml, (OT*)out, o_stride, n_heads * maps, vdim, splits, out_scale,
+                                           Gate{gate, gate_stride}));
                 TI_CHECK_LAUNCH("attn_window_merge");
             }
             return 0;
@@ -970,9 +1027,11 @@ extern "C" int ti_attn_window_decode(const void* q, long long q_stride, void* ou
 }
 
 // The merge alone, for partial results that another kernel left (the tensor-core kernel for single tokens): part_o
-// [n_seq, virtual heads, splits, vdim], part_ml [n_seq, virtual heads, splits, 2] -> out [n_seq, virtual heads * vdim].
+// [n_seq, virtual heads, splits, vdim], part_ml [n_seq, virtual heads, splits, 2] -> out [n_seq, virtual heads * vdim],
+// times sigmoid(gate) where gate ([n_seq, virtual heads * vdim] of the engine's type) is given.
 extern "C" int ti_attn_window_merge(const float* part_o, const float* part_ml, void* out, long long o_stride, int out_f32, int n_seq,
-                                    int n_virtual, int vdim, int splits, int mode, float out_scale, int dtype, cudaStream_t stream) {
+                                    int n_virtual, int vdim, int splits, int mode, float out_scale, const void* gate,
+                                    long long gate_stride, int dtype, cudaStream_t stream) {
     if (n_seq == 0) return 0;
     TI_REQUIRE(n_seq > 0 && n_seq <= 65535 && n_virtual > 0 && vdim > 0 && splits >= 1 && part_o && part_ml, "attn_window_merge: bad sizes");
     TI_REQUIRE(mode == 0 || mode == 1, "attn_window_merge: unknown mode %d", mode);
@@ -980,8 +1039,8 @@ extern "C" int ti_attn_window_merge(const float* part_o, const float* part_ml, v
         using T = decltype(t);
         auto go = [&](auto ot, auto md) -> int {
             using OT = decltype(ot);
-            TI_CUDA(ti_launch_class<4>(attn_window_merge_kernel<OT, decltype(md)::value>, dim3(n_virtual, n_seq), dim3(64), 0, stream, part_o,
-                                       part_ml, (OT*)out, o_stride, n_virtual, vdim, splits, out_scale));
+            TI_CUDA(ti_launch_class<4>(attn_window_merge_kernel<T, OT, decltype(md)::value>, dim3(n_virtual, n_seq), dim3(64), 0, stream, part_o,
+                                       part_ml, (OT*)out, o_stride, n_virtual, vdim, splits, out_scale, Gate{gate, gate_stride}));
             TI_CHECK_LAUNCH("attn_window_merge");
             return 0;
         };

@@ -1,10 +1,10 @@
-// A float32 residual stream between sublayers that are normed on the way in AND on the way out.
+// A float32 residual stream between sublayers that are normed on the way out, and on the way in or not.
 //
-// A layer of such a design does  h <- h + n_post(f(n_pre(h)))  per sublayer f, with
+// A layer of such a design does  h <- h + n_post(f(n_pre(h)))  or  h <- h + n_post(f(h))  per sublayer f, with
 // n(v) = v * rsqrt(mean(v^2) + eps) * w.  The sublayer's output y (engine type) stays pending
 // until the next reader of the stream: this kernel forms n_post(y), adds it to the float32 row of
-// h without rounding, writes the row back, and norms the new row for the next sublayer, all in
-// one pass (one block per row).  With `rows` it works on the gathered rows only and leaves h
+// h without rounding, writes the row back, and norms the new row for the next sublayer (without a
+// norm on the way in: rounds it to the engine's type), all in one pass (one block per row).  With `rows` it works on the gathered rows only and leaves h
 // alone (the head's rows).  A norm weight is float32, one number (stride 0) or one per channel
 // (stride 1).
 #include "common.cuh"
@@ -43,9 +43,10 @@ __global__ void post_norm_add_norm_kernel(float* __restrict__ h, const T* __rest
         if (!ok) x = 0.f;
         row[i] = x;
         if (write_back && y) h[base + i] = x;
+        if (out && !w_pre) out[(size_t)r * H + i] = from_f32<T>(x);
         ss = fmaf(x, x, ss);
     }
-    if (!out) return;
+    if (!out || !w_pre) return;
     const float inv = rsqrtf(block_sum(ss, red) / (float)H + eps);
     for (int i = threadIdx.x; i < H; i += blockDim.x)
         out[(size_t)r * H + i] = from_f32<T>(row[i] * inv * w_pre[(size_t)i * pre_stride]);
@@ -54,7 +55,7 @@ __global__ void post_norm_add_norm_kernel(float* __restrict__ h, const T* __rest
 }  // namespace
 
 // h: float32 [M, H].  y: [M, H] of the engine's type or null (nothing pending).  w_post / w_pre: float32, one number
-// (stride 0) or H (stride 1).  rows: null (every row, R == M) or R row indices.  out: [R, H] of the engine's type or
+// (stride 0) or H (stride 1); w_pre null: out takes the rounded sum itself.  rows: null (every row, R == M) or R row indices.  out: [R, H] of the engine's type or
 // null (only the sum is wanted).  write_back: store the sum into h.
 extern "C" int ti_post_norm_add_norm(float* h, const void* y, const float* w_post, int post_stride, const int* rows,
                                      const float* w_pre, int pre_stride, void* out, int R, int H, int M, float eps,
@@ -64,7 +65,6 @@ extern "C" int ti_post_norm_add_norm(float* h, const void* y, const float* w_pos
     TI_REQUIRE(rows || R == M, "post_norm_add_norm: without row indices every row is taken (R=%d, M=%d)", R, M);
     TI_REQUIRE(!(rows && write_back), "post_norm_add_norm: gathered rows are not written back");
     TI_REQUIRE(!y || w_post, "post_norm_add_norm: a pending output needs its norm weight");
-    TI_REQUIRE(!out || w_pre, "post_norm_add_norm: normed rows need a norm weight");
     TI_REQUIRE((post_stride == 0 || post_stride == 1) && (pre_stride == 0 || pre_stride == 1), "post_norm_add_norm: weight strides are 0 or 1");
     const size_t smem = (size_t)(H + 33) * sizeof(float);
     TI_REQUIRE(smem <= 200 * 1024, "post_norm_add_norm: rows of %d elements do not fit shared memory", H);

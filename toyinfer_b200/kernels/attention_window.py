@@ -56,13 +56,16 @@ def prepare(qkv: torch.Tensor, bias: Optional[torch.Tensor], q_w: Optional[torch
 
 
 def head_prepare(qkv: torch.Tensor, bias: Optional[torch.Tensor], q_w: Optional[torch.Tensor], k_w: Optional[torch.Tensor], eps: float,
-                 tables, pairing: str, n_heads: int, n_kv: int, dim: int, vdim: int, mem, batch) -> None:
+                 tables, pairing: str, n_heads: int, n_kv: int, dim: int, vdim: int, mem, batch, temperature=None,
+                 blend: Optional[torch.Tensor] = None, mix: float = 0.0) -> None:
     """As ``prepare`` for one score map and norms per head: qkv [M, >= heads * dim + kv_heads * (dim + vdim)]; adds ``bias``
     (float32, q, k and v's length), norms every head of q over its ``dim`` elements with the weight ``q_w`` (float32 [dim],
     the same for all heads; None: no norm) and every head of k with ``k_w``, rotates the first ``rot`` elements of every head
     of q and k (``tables`` = (cos, sin, rot) or None; ``pairing`` "half": element e turns with e + rot / 2, "neighbours":
-    2e with 2e + 1), leaves the queries in place and stores keys and values in ``mem``."""
-    _need_cuda(qkv, bias, q_w, k_w, what="attention_window.head_prepare")
+    2e with 2e + 1), leaves the queries in place and stores keys and values in ``mem``.  ``temperature`` = (coef, every): the
+    query at position p is multiplied by 1 + coef ln(floor((p + 1) / every) + 1).  ``blend`` [M, kv_heads * vdim] (another
+    layer's values of the same tokens, rows may be strided): a value v becomes (1 - mix) v + mix blend."""
+    _need_cuda(qkv, bias, q_w, k_w, blend, what="attention_window.head_prepare")
     M, N = qkv.shape
     nq, nk, nv = n_heads * dim, n_kv * dim, n_kv * vdim
     if N < nq + nk + nv or qkv.stride(1) != 1:
@@ -70,6 +73,11 @@ def head_prepare(qkv: torch.Tensor, bias: Optional[torch.Tensor], q_w: Optional[
     for t, n in ((bias, nq + nk + nv), (q_w, dim), (k_w, dim)):
         if t is not None and (t.dtype != torch.float32 or t.numel() != n or not t.is_contiguous()):
             raise KernelError("attention_window.head_prepare: biases and norm weights must be dense float32")
+    coef, every = temperature if temperature is not None else (0.0, 0)
+    if temperature is not None and int(every) < 1:
+        raise KernelError(f"attention_window.head_prepare: a temperature that grows every {every} positions")
+    if blend is not None and (tuple(blend.shape) != (M, nv) or blend.dtype != qkv.dtype or blend.stride(1) != 1):
+        raise KernelError(f"attention_window.head_prepare: values to blend in must be [{M}, {nv}] of the projection's type")
     if pairing not in ("half", "neighbours"):
         raise KernelError(f"attention_window.head_prepare: unknown pairing {pairing!r}")
     cos = sin = None
@@ -81,10 +89,11 @@ def head_prepare(qkv: torch.Tensor, bias: Optional[torch.Tensor], q_w: Optional[
             raise KernelError("attention_window.head_prepare: rotary tables must be float32 [positions, rot / 2] with rot <= dim")
         if batch.max_pos_after > max_pos:
             raise KernelError(f"attention_window.head_prepare: position {batch.max_pos_after - 1} is beyond the rotary tables' {max_pos}")
-    _call(_fn("ti_attn_head_prepare", [P, L, P, P, P, F, P, P, I, I, I, P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, P]),
+    _call(_fn("ti_attn_head_prepare", [P, L, P, P, P, F, P, P, I, I, I, P, P, P, P, P, P, I, I, I, I, I, I, I, I, F, I, P, L, F, I, P]),
           _ptr(qkv), qkv.stride(0), _ptr(bias), _ptr(q_w), _ptr(k_w), float(eps), _ptr(cos), _ptr(sin), int(rot),
           1 if pairing == "neighbours" else 0, int(max_pos), _ptr(batch.tok_pos), _ptr(batch.tok_seq), _ptr(batch.seq_slot),
           *_pages(mem, qkv.dtype, n_kv, dim, vdim, "attention_window.head_prepare"), M, n_heads, n_kv, dim, vdim,
+          float(coef), int(every), _ptr(blend), blend.stride(0) if blend is not None else 0, float(mix),
           _code(qkv, "attention_window"), _stream())
 
 
@@ -123,12 +132,13 @@ def attend(q: torch.Tensor, maps: int, vdim: int, mem, scale: float, window: int
            r1: Optional[torch.Tensor] = None, r2: Optional[torch.Tensor] = None, pb: Optional[torch.Tensor] = None,
            out_f32: bool = False, k: Optional[torch.Tensor] = None, v: Optional[torch.Tensor] = None,
            table: Optional[torch.Tensor] = None, keep_first: int = 0, out_scale: float = 1.0,
-           out: Optional[torch.Tensor] = None) -> torch.Tensor:
+           out: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None) -> torch.Tensor:
     """q [M, heads * maps, dim] (prepared) over the keys and values that ``mem`` holds, the step's own included ->
     [M, heads * maps * vdim] (float32 with ``out_f32``, else q's type), times ``out_scale`` before the rounding; ``out``
     (that shape, rows may be strided: columns of a wider buffer) takes the result when given.  Key j is visible to query
     i when 0 <= i - j < window, or when j <= i and j < ``keep_first`` (a sequence's first positions, which a window
-    would hide, stay visible).  r1, r2: float32 [heads], the score loses r1 ln(1 + r2 (i - j)); pb: float32 [heads], added to
+    would hide, stay visible).  ``gate`` [M, heads * maps * vdim] (q's type, rows may be strided): every element of the result
+    is multiplied by sigmoid(gate).  r1, r2: float32 [heads], the score loses r1 ln(1 + r2 (i - j)); pb: float32 [heads], added to
     the score under the sigmoid.  mode: "softmax" or "sigmoid" (weights not normalised over the keys).
     k [M, kv_heads * maps * dim], v [M, kv_heads * vdim]: the step's own keys and values as ``prepare`` left them, and
     ``table`` (``distance_table``; sigmoid mode) let prompts and pieces run on the tensor cores: bfloat16, keys and values
@@ -136,7 +146,7 @@ def attend(q: torch.Tensor, maps: int, vdim: int, mem, scale: float, window: int
     Single tokens (a step in which every sequence goes on by one) run on the tensor-core decode kernel
     (csrc/attn_decode_mma.cu) in bfloat16 where a key row, all maps together, is as long as a value row (64 or 128), with
     the same rounding of the weights; else on the CUDA-core kernel of csrc/attn_window.cu."""
-    _need_cuda(q, r1, r2, pb, what="attention_window")
+    _need_cuda(q, r1, r2, pb, gate, what="attention_window")
     M, HV, dim = q.shape
     if HV % maps or q.stride(2) != 1 or q.stride(1) != dim:
         raise KernelError("attention_window: heads of a token must be dense")
@@ -153,6 +163,9 @@ def attend(q: torch.Tensor, maps: int, vdim: int, mem, scale: float, window: int
     o_dtype = torch.float32 if out_f32 else q.dtype
     if out is not None and (tuple(out.shape) != (M, HV * vdim) or out.dtype != o_dtype or out.stride(1) != 1 or not out.is_cuda):
         raise KernelError("attention_window: the result's place must be [tokens, heads * maps * vdim] of the result's type with dense rows")
+    if gate is not None and (tuple(gate.shape) != (M, HV * vdim) or gate.dtype != q.dtype or gate.stride(1) != 1):
+        raise KernelError(f"attention_window: the gate must be [{M}, {HV * vdim}] of the queries' type with dense rows")
+    gated = (_ptr(gate), gate.stride(0) if gate is not None else 0)
     if batch.mode == "extend" and tensor_cores and q.dtype == torch.bfloat16 and maps * dim == vdim and vdim in (64, 128) \
             and dim % 8 == 0 and mem.page_size == 64 and (maps == 1 if mode == "sigmoid" else (r1 is None and pb is None)) \
             and q.stride(0) % 2 == 0 and q.data_ptr() % 4 == 0:
@@ -170,14 +183,14 @@ def attend(q: torch.Tensor, maps: int, vdim: int, mem, scale: float, window: int
         use_table = mode == "sigmoid" and table is not None
         if use_table and (table.dtype != torch.float32 or table.dim() != 2 or table.shape[0] != H or not table.is_contiguous()):
             raise KernelError("attention_window: the distance table must be dense float32 [heads, far + 1]")
-        _call(_fn("ti_attn_decode_mma_scored", [P, L, P, P, P, I, I, I, I, P, P, I, I, I, I, I, F, I, I, P, P, P, P, I, I, F, I, P, L, I, P, P, I, P]),
+        _call(_fn("ti_attn_decode_mma_scored", [P, L, P, P, P, I, I, I, I, P, P, I, I, I, I, I, F, I, I, P, P, P, P, I, I, F, I, P, L, I, P, P, P, L, I, P]),
               _ptr(q), q.stride(0), pages[0], pages[1], pages[2], pages[3], pages[4], 0, pages[5], _ptr(batch.seq_slot),
               _ptr(batch.seq_len), M, H, G, maps, vdim, float(scale), int(window), MODES[mode], _ptr(r1), _ptr(r2), _ptr(pb),
               _ptr(table) if use_table else None, table.shape[1] - 1 if use_table else 0, keep_first, float(out_scale), splits,
-              _ptr(out), out.stride(0), 1 if out_f32 else 0, _ptr(part_o), _ptr(part_ml), code, _stream())
+              _ptr(out), out.stride(0), 1 if out_f32 else 0, _ptr(part_o), _ptr(part_ml), *gated, code, _stream())
         if splits > 1:
-            _call(_fn("ti_attn_window_merge", [P, P, P, L, I, I, I, I, I, I, F, I, P]), _ptr(part_o), _ptr(part_ml), _ptr(out), out.stride(0),
-                  1 if out_f32 else 0, M, HV, vdim, splits, MODES[mode], float(out_scale), code, _stream())
+            _call(_fn("ti_attn_window_merge", [P, P, P, L, I, I, I, I, I, I, F, P, L, I, P]), _ptr(part_o), _ptr(part_ml), _ptr(out), out.stride(0),
+                  1 if out_f32 else 0, M, HV, vdim, splits, MODES[mode], float(out_scale), *gated, code, _stream())
         return out
     if out is None:
         out = torch.zeros((M, HV * vdim), dtype=o_dtype, device=q.device)
@@ -188,28 +201,29 @@ def attend(q: torch.Tensor, maps: int, vdim: int, mem, scale: float, window: int
         if splits > 1:
             part_o = torch.empty((M, HV, splits, vdim), dtype=torch.float32, device=q.device)
             part_ml = torch.empty((M, HV, splits, 2), dtype=torch.float32, device=q.device)
-        _call(_fn("ti_attn_window_decode", [P, L, P, L, I, P, P, I, P, P, P, I, I, I, P, P, P, I, I, I, I, I, F, I, I, F, I, I, P, P, I, P]),
+        _call(_fn("ti_attn_window_decode", [P, L, P, L, I, P, P, I, P, P, P, I, I, I, P, P, P, I, I, I, I, I, F, I, I, F, I, I, P, P, P, L, I, P]),
               _ptr(q), q.stride(0), _ptr(out), out.stride(0), 1 if out_f32 else 0, _ptr(batch.seq_len), _ptr(batch.seq_slot), M, *pages,
               _ptr(r1), _ptr(r2), _ptr(pb), H, G, maps, dim, vdim, float(scale), int(window), keep_first, float(out_scale), MODES[mode], splits,
-              _ptr(part_o), _ptr(part_ml), code, _stream(), launches=2 if splits > 1 else 1)
+              _ptr(part_o), _ptr(part_ml), *gated, code, _stream(), launches=2 if splits > 1 else 1)
         return out
     if tensor_cores and q.dtype == torch.bfloat16 and dim in (64, 128) and vdim in (64, 128) and k is not None and v is not None \
             and mem.page_size == 64 and scale > 0 and (mode == "softmax" or table is not None) and (mode == "sigmoid" or r1 is None) \
             and all(t.stride(0) % 8 == 0 and t.data_ptr() % 16 == 0 and t.stride(-1) == 1 for t in (q, k, v)) \
+            and (gate is None or (gate.stride(0) % 8 == 0 and gate.data_ptr() % 16 == 0)) \
             and out.stride(0) % (4 if out_f32 else 8) == 0 and out.data_ptr() % 16 == 0:
         if table is not None and (table.dtype != torch.float32 or table.dim() != 2 or table.shape[0] != H or not table.is_contiguous()):
             raise KernelError("attention_window: the distance table must be dense float32 [heads, far + 1]")
         start = batch.mode == "start"
-        _call(_fn("ti_attn_window_tc", [P, P, P, P, L, L, L, L, I, P, P, P, I, I, I, I, I, I, I, I, F, I, I, P, P, P, I, I, I, P, I, I, F, P]),
+        _call(_fn("ti_attn_window_tc", [P, P, P, P, L, L, L, L, I, P, P, P, I, I, I, I, I, I, I, I, F, I, I, P, P, P, I, I, I, P, I, I, F, P, L, P]),
               _ptr(q), _ptr(k), _ptr(v), _ptr(out), q.stride(0), k.stride(0), v.stride(0), out.stride(0), 1 if out_f32 else 0,
               _ptr(batch.cu_new), None if start else _ptr(batch.seq_start), _ptr(batch.seq_slot), batch.n_seq, batch.max_new, M, H, G,
               maps, dim, vdim, float(scale), int(window), MODES[mode], *pages, _ptr(table) if mode == "sigmoid" else None,
-              table.shape[1] - 1 if (mode == "sigmoid" and table is not None) else 0, keep_first, float(out_scale), _stream())
+              table.shape[1] - 1 if (mode == "sigmoid" and table is not None) else 0, keep_first, float(out_scale), *gated, _stream())
         return out
-    _call(_fn("ti_attn_window", [P, L, P, L, I, P, P, P, I, I, P, P, P, I, I, I, P, P, P, I, I, I, I, I, F, I, I, F, I, I, P]),
+    _call(_fn("ti_attn_window", [P, L, P, L, I, P, P, P, I, I, P, P, P, I, I, I, P, P, P, I, I, I, I, I, F, I, I, F, I, P, L, I, P]),
           _ptr(q), q.stride(0), _ptr(out), out.stride(0), 1 if out_f32 else 0, _ptr(batch.cu_new), _ptr(batch.seq_start),
           _ptr(batch.seq_slot), batch.n_seq, batch.max_new, *pages, _ptr(r1), _ptr(r2), _ptr(pb), H, G, maps, dim, vdim, float(scale),
-          int(window), keep_first, float(out_scale), MODES[mode], code, _stream())
+          int(window), keep_first, float(out_scale), MODES[mode], *gated, code, _stream())
     return out
 
 

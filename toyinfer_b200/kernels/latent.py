@@ -94,6 +94,14 @@ def plan(n_seq: int, n_heads: int, window: int, plan_len: int, device) -> int:
     return decode_splits(n_seq, n_heads, heads_per_block(n_heads, True), span, sm_count(device))
 
 
+def _gate(gate: Optional[torch.Tensor], M: int, n_heads: int, dtype, what: str):
+    if gate is None:
+        return (None, 0)
+    if tuple(gate.shape) != (M, n_heads) or gate.dtype != dtype or gate.stride(1) != 1 or not gate.is_cuda:
+        raise KernelError(f"{what}: the gate must be [{M}, {n_heads}] of the queries' type with dense rows, on the device")
+    return (_ptr(gate), gate.stride(0))
+
+
 def prompt_heads(plain: int, rot: int, vdim: int) -> int:
     """The head size (64 or 128) at which a step of whole prompts runs as plain multi-head attention on the tensor cores,
     or 0 when the heads do not fit."""
@@ -102,10 +110,11 @@ def prompt_heads(plain: int, rot: int, vdim: int) -> int:
 
 
 def attention_prompt(q: torch.Tensor, lat: torch.Tensor, w_ukv: torch.Tensor, vdim: int, rank: int, rot: int, scale: float,
-                     window: int, sink: Optional[torch.Tensor], batch, D: int) -> torch.Tensor:
+                     window: int, sink: Optional[torch.Tensor], batch, D: int, gate: Optional[torch.Tensor] = None) -> torch.Tensor:
     """Every sequence starts at position 0, bfloat16: keys and values per head are formed from the step's rows by one product
     with w_ukv = [Wuk; Wuv], packed beside the queries into heads of D elements, and a multi-head attention over the step's own
-    tokens runs on the tensor cores.  Returns [M, heads * D]: head h's value in its first ``vdim`` elements, zeros after."""
+    tokens runs on the tensor cores.  Returns [M, heads * D]: head h's value in its first ``vdim`` elements, zeros after.
+    ``gate`` [M, heads] (rows may be strided): head h's value times sigmoid(gate_h)."""
     from . import linear
     from .lib import library
     M, nh, hd = q.shape
@@ -115,9 +124,9 @@ def attention_prompt(q: torch.Tensor, lat: torch.Tensor, w_ukv: torch.Tensor, vd
     Kp, Vp, out = torch.empty_like(Qp), torch.empty_like(Qp), torch.empty_like(Qp)
     _call(_fn("ti_latent_pack", [P, L, P, P, P, P, P, I, I, I, I, I, I, I, I, P]), _ptr(q), q.stride(0), _ptr(ku), _ptr(lat),
           _ptr(Qp), _ptr(Kp), _ptr(Vp), M, nh, plain, rot, vdim, rank, D, _code(q, "latent_pack"), _stream())
-    _call(_fn("ti_attn_prefill_tc_sink", [P, P, P, P, L, L, L, L, P, I, I, I, I, I, I, F, I, P, P]),
+    _call(_fn("ti_attn_prefill_tc_sink", [P, P, P, P, L, L, L, L, P, I, I, I, I, I, I, F, I, P, P, L, P]),
           _ptr(Qp), _ptr(Kp), _ptr(Vp), _ptr(out), nh * D, nh * D, nh * D, nh * D, _ptr(batch.cu_new), batch.n_seq, batch.max_new,
-          M, nh, nh, D, float(scale), int(window), _ptr(sink), _stream())
+          M, nh, nh, D, float(scale), int(window), _ptr(sink), *_gate(gate, M, nh, q.dtype, "latent_attention"), _stream())
     return out.view(M, nh * D)
 
 
@@ -139,11 +148,11 @@ def single_eligible(q: torch.Tensor, rank: int, rot: int, batch, mem) -> bool:
 
 def attention_single(d: torch.Tensor, q: torch.Tensor, rank: int, rot: int, norm_w: torch.Tensor, eps: float, tables,
                      uk: torch.Tensor, uv: torch.Tensor, vdim: int, scale: float, window: int, sink: Optional[torch.Tensor],
-                     batch, mem) -> torch.Tensor:
+                     batch, mem, gate: Optional[torch.Tensor] = None) -> torch.Tensor:
     """A step in which every sequence brings one token, bfloat16, in three launches: the token's row (normed, rotated, stored)
     together with its queries' way into the latent space; the attention over the cached rows on the tensor cores, a
     sequence's keys split over blocks; the splits' merge together with the way out through uv.  d[M, rank + rot] and
-    q[M, heads, plain + rot] are the projection's output as it is -> [M, heads * vdim]."""
+    q[M, heads, plain + rot] are the projection's output as it is -> [M, heads * vdim]; ``gate`` as in attention_prompt."""
     _need_cuda(d, q, norm_w, uk, uv, sink, what="latent_attention")
     M, nh, hd = q.shape
     plain, W = hd - rot, rank + rot
@@ -165,17 +174,18 @@ def attention_single(d: torch.Tensor, q: torch.Tensor, rank: int, rot: int, norm
     part_o = torch.empty((M, nh, splits, rank), dtype=torch.float32, device=q.device)
     part_ml = torch.empty((M, nh, splits, 2), dtype=torch.float32, device=q.device)
     o = torch.empty((M, nh * vdim), dtype=q.dtype, device=q.device)
-    _call(_fn("ti_latent_decode", [P, P, P, P, P, I, I, I, I, F, I, P, P, P, I, I, I, I, I, P, P, P, P, L, I, P]),
+    _call(_fn("ti_latent_decode", [P, P, P, P, P, I, I, I, I, F, I, P, P, P, I, I, I, I, I, P, P, P, P, L, I, P, L, P]),
           _ptr(qa), _ptr(lat), _ptr(batch.cu_new), _ptr(batch.seq_start), _ptr(batch.seq_slot), batch.n_seq, nh, rank, rot,
           float(scale), int(window), _ptr(sink), *_pages(mem), splits, _ptr(part_o), _ptr(part_ml), _ptr(uv), _ptr(o), o.stride(0),
-          vdim, _stream(), launches=2)
+          vdim, *_gate(gate, M, nh, q.dtype, "latent_attention"), _stream(), launches=2)
     return o
 
 
 def attention(q: torch.Tensor, lat: torch.Tensor, uk: torch.Tensor, uv: torch.Tensor, vdim: int, rank: int, rot: int,
-              scale: float, window: int, sink: Optional[torch.Tensor], batch, mem) -> torch.Tensor:
+              scale: float, window: int, sink: Optional[torch.Tensor], batch, mem, gate: Optional[torch.Tensor] = None) -> torch.Tensor:
     """q[M, heads, plain + rot] (rotated part already rotated), the step's rows lat[M, rank + rot], uk[heads * plain, rank],
-    uv[heads * vdim, rank] -> [M, heads * vdim].  Keys at positions below a sequence's start come from ``mem``."""
+    uv[heads * vdim, rank] -> [M, heads * vdim].  Keys at positions below a sequence's start come from ``mem``;
+    ``gate`` as in attention_prompt."""
     _need_cuda(q, lat, uk, uv, sink, what="latent_attention")
     M, nh, hd = q.shape
     plain, W = hd - rot, rank + rot
@@ -204,6 +214,6 @@ def attention(q: torch.Tensor, lat: torch.Tensor, uk: torch.Tensor, uv: torch.Te
           batch.max_new, nh, hb, rank, rot, float(scale), int(window), _ptr(sink), *_pages(mem), splits, _ptr(part_o),
           _ptr(part_ml), M, code, _stream(), launches=2 if splits > 1 else 1)
     o = torch.empty((M, nh * vdim), dtype=q.dtype, device=q.device)
-    _call(_fn("ti_latent_expand", [P, P, P, L, I, I, I, I, I, P]), _ptr(ol), _ptr(uv), _ptr(o), o.stride(0), M, nh, vdim, rank,
-          code, _stream())
+    _call(_fn("ti_latent_expand", [P, P, P, L, I, I, I, I, P, L, I, P]), _ptr(ol), _ptr(uv), _ptr(o), o.stride(0), M, nh, vdim, rank,
+          *_gate(gate, M, nh, q.dtype, "latent_attention"), code, _stream())
     return o

@@ -95,10 +95,10 @@ def _norm_weight(w: Optional[torch.Tensor], H: int, what: str) -> int:
 
 
 def post_norm_add_norm(h: torch.Tensor, pending: Optional[PostNormed], weight: Optional[torch.Tensor], eps: float,
-                       out_dtype: torch.dtype, rows: Optional[torch.Tensor] = None) -> Optional[torch.Tensor]:
+                       out_dtype: torch.dtype, rows: Optional[torch.Tensor] = None, rounded: bool = False) -> Optional[torch.Tensor]:
     """h (float32 [M, H]) takes rmsnorm(pending.y) * pending.weight in place (without ``rows``); returns
-    rmsnorm(h) * weight in ``out_dtype`` (None when ``weight`` is None: only the sum is wanted).  With ``rows`` only those
-    rows are summed and normed and h is left as it is."""
+    rmsnorm(h) * weight in ``out_dtype`` (when ``weight`` is None: with ``rounded`` the sum itself in that type, else None).
+    With ``rows`` only those rows are summed and normed and h is left as it is."""
     y = pending.y if pending is not None else None
     wp = pending.weight if pending is not None else None
     _need_cuda(h, y, wp, weight, rows, what="post_norm_add_norm")
@@ -115,7 +115,7 @@ def post_norm_add_norm(h: torch.Tensor, pending: Optional[PostNormed], weight: O
     if rows is not None:
         _i32(rows, "post_norm_add_norm rows")
         R = rows.numel()
-    out = torch.empty((R, H), dtype=out_dtype, device=h.device) if weight is not None else None
+    out = torch.empty((R, H), dtype=out_dtype, device=h.device) if weight is not None or rounded else None
     _call(_fn("ti_post_norm_add_norm", [P, P, P, I, P, P, I, P, I, I, I, F, I, I, P]),
           _ptr(h), _ptr(y), _ptr(wp), sp, _ptr(rows), _ptr(weight), sw, _ptr(out), R, H, M,
           float(pending.eps if weight is None and pending is not None else eps), 0 if rows is not None else 1,

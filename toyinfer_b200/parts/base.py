@@ -29,6 +29,8 @@ Families and what each must provide:
                     agrees.  ``shared`` is a dict that lives for one
                     step and belongs to the schedule entry that owns ``mem``; an
                     entry that borrows another entry's memory gets the owner's dict.
+                    Its item ``"step"`` is one dict for all entries of the step, in which a
+                    layer leaves per-token tensors that later layers read.
                     When it holds a list ``"deferred"``, later entries still read
                     ``mem``: a write that would destroy what they read is appended
                     there as a callable instead of being done.

@@ -149,7 +149,8 @@ class DecoderModel(Part):
         with ranged(batch, "embed"):
             h = self.embedding.forward(batch.token_ids)
         delta = None
-        shared: List[dict] = [dict() for _ in self.schedule]
+        carried: dict = {}         # what a layer leaves for later layers of this step, by name
+        shared: List[dict] = [{"step": carried} for _ in self.schedule]
         owners = [i if e.memory_of is None else e.memory_of for i, e in enumerate(self.schedule)]
         last_use = {o: i for i, o in enumerate(owners)}
         for o, last in last_use.items():

@@ -129,6 +129,11 @@ class WideScalarRMSNorm(Norm):
         """y as something that passes this norm before it is added to the stream."""
         return wide.PostNormed(y, self.weight, self.eps)
 
+    def read_forward(self, h: torch.Tensor, delta) -> torch.Tensor:
+        """h takes what is pending; returns the sum itself in the engine's type (for a sublayer that reads the stream as it is)."""
+        self._check(delta)
+        return wide.post_norm_add_norm(h, delta, None, self.eps, self.out_dtype, rounded=True)
+
     def _check(self, delta) -> None:
         if delta is not None and not isinstance(delta, wide.PostNormed):
             raise ValueError("a stream with normed sublayer outputs takes what a norm's pending() made, nothing else")

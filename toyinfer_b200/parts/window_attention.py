@@ -27,7 +27,14 @@ the token's position, in the pairing that the position encoding names; key j is 
 0 <= i - j < window, or when j <= i and j < keep_first: the first ``keep_first`` positions of a sequence stay visible to
 every later query, at their own positions; softmax over the visible keys.  Its result may be scaled and placed in the
 columns of a wider buffer, and its projections' rows handed out, so that it can stand beside another mixer
-(parts/side_by_side.py).
+(parts/side_by_side.py).  ``biases`` "qkv": on the first three projections only.  Further options, each off by default:
+
+  * ``temperature`` {coef, every}: the normed query at position p is multiplied by 1 + coef ln(floor((p + 1) / every) + 1);
+  * ``values`` "first" / "blended": the layer's own values of the step's tokens are left for later layers, or are blended with
+    those, v <- (1 - lambda) v + lambda v_first, before they are stored (lambda one number per layer, ``vmix``); v_first
+    needs no memory, since only the same token's is read;
+  * ``gate``: the heads side by side are multiplied, element by element, by sigmoid(Wg x) before the output projection; the
+    gate's rows ride with the q, k, v projection and the attention's last kernel applies them.
 
 Keys and values of all positions live in the cache; a step first stores its own, then attends over the pages,
 whatever mix of new and cached tokens it brings.  Only the last ``window`` positions are ever read.
@@ -211,21 +218,31 @@ class KeptWindowAttention(_WindowAttention):
     """Softmax attention under a sliding window that keeps the first ``keep_first`` positions visible (see the module's text)."""
 
     def __init__(self, ctx: BuildContext, prefix: str, n_heads: int, n_kv_heads: int, dim: int, vdim: int, scale: float,
-                 window: int, eps: float, keep_first: int = 0, position: Optional[str] = None, biases: bool = True,
-                 head_norm=True, names: Optional[Dict[str, str]] = None):
+                 window: int, eps: float, keep_first: int = 0, position: Optional[str] = None, biases=True,
+                 head_norm=True, temperature: Optional[dict] = None, values: Optional[str] = None, gate: bool = False,
+                 names: Optional[Dict[str, str]] = None):
         self._sizes(ctx, prefix, n_heads, n_kv_heads, dim, vdim, scale, window, eps)
         if int(keep_first) < 0:
             raise ValueError(f"attention at {prefix!r}: {keep_first} kept first positions")
         self.keep_first = int(keep_first) if self.window > 0 else 0
         if head_norm not in (True, False, "unit"):
             raise ValueError(f"attention at {prefix!r}: head_norm is True, False or 'unit', got {head_norm!r}")
-        self.biases, self.head_norm = bool(biases), head_norm
+        if biases not in (True, False, "qkv"):
+            raise ValueError(f"attention at {prefix!r}: biases is True, False or 'qkv', got {biases!r}")
+        if values not in (None, "first", "blended"):
+            raise ValueError(f"attention at {prefix!r}: values is None, 'first' or 'blended', got {values!r}")
+        self.biases, self.head_norm = biases, head_norm
+        self.temperature = (float(temperature["coef"]), int(temperature["every"])) if temperature else None
+        if self.temperature is not None and self.temperature[1] < 1:
+            raise ValueError(f"attention at {prefix!r}: a temperature that grows every {temperature['every']} positions")
+        self.values, self.gate = values, bool(gate)
+        self.lam = 0.0
         self.position = None
         if position is not None:
             if position not in ctx.positions:
                 raise ValueError(f"attention at {prefix!r} names position encoding {position!r}, which the model does not have")
             self.position = ctx.positions[position]
-        n = {"q": "q", "k": "k", "v": "v", "o": "o", "q_norm": "q.norm", "k_norm": "k.norm", "bias": ".b"}
+        n = {"q": "q", "k": "k", "v": "v", "o": "o", "g": "g", "vmix": "vmix", "q_norm": "q.norm", "k_norm": "k.norm", "bias": ".b"}
         n.update(names or {})
         self.n = n
         self.w_qkv = self.w_o = self.b_qkv = self.b_o = self.q_w = self.k_w = None
@@ -235,7 +252,8 @@ class KeptWindowAttention(_WindowAttention):
 
     @property
     def n_in(self) -> int:
-        return self.n_heads * self.dim + self.n_kv * (self.dim + self.vdim)
+        n = self.n_heads * self.dim + self.n_kv * (self.dim + self.vdim) + (self.n_heads * self.vdim if self.gate else 0)
+        return n + (-n % 8 if self.gate else 0)
 
     @property
     def n_out(self) -> int:
@@ -248,7 +266,12 @@ class KeptWindowAttention(_WindowAttention):
              self._name("v"): ParamSpec((G * vd, self.hidden), std=0.05), self._name("o"): ParamSpec((self.hidden, H * vd), std=0.05)}
         if self.biases:
             for k, rows in (("q", H * d), ("k", G * d), ("v", G * vd), ("o", self.hidden)):
-                s[self._name(k, True)] = small((rows,), init="normal", std=0.1)
+                if k != "o" or self.biases is True:
+                    s[self._name(k, True)] = small((rows,), init="normal", std=0.1)
+        if self.gate:
+            s[self._name("g")] = ParamSpec((H * vd, self.hidden), std=0.1)
+        if self.values == "blended":
+            s[self._name("vmix")] = small((), init="normal", mean=0.4, std=0.1)
         if self.head_norm is True:
             s[self._name("q_norm")] = small((d,), init="one_plus_normal", std=0.1)
             s[self._name("k_norm")] = small((d,), init="one_plus_normal", std=0.1)
@@ -257,11 +280,18 @@ class KeptWindowAttention(_WindowAttention):
     def bind(self, tensors: Dict[str, torch.Tensor]) -> None:
         t = lambda name: tensors.pop(name)
         f32 = lambda name: t(name).to(torch.float32).contiguous()
-        self.w_qkv = torch.cat([t(self._name(k)) for k in ("q", "k", "v")], dim=0).contiguous()
+        parts = [t(self._name(k)) for k in (("q", "k", "v", "g") if self.gate else ("q", "k", "v"))]
+        spare = self.n_in - sum(p.shape[0] for p in parts)
+        if spare:                   # a row of results that is a multiple of 16 bytes long
+            parts.append(torch.zeros((spare, self.hidden), dtype=parts[0].dtype, device=parts[0].device))
+        self.w_qkv = torch.cat(parts, dim=0).contiguous()
         self.w_o = t(self._name("o")).contiguous()
         if self.biases:
             self.b_qkv = torch.cat([f32(self._name(k, True)) for k in ("q", "k", "v")]).contiguous()
-            self.b_o = f32(self._name("o", True))
+            if self.biases is True:
+                self.b_o = f32(self._name("o", True))
+        if self.values == "blended":
+            self.lam = float(t(self._name("vmix")).to(torch.float32))
         if self.head_norm == "unit":
             self.q_w = self.k_w = torch.ones(self.dim, dtype=torch.float32, device=self.w_o.device)
         elif self.head_norm:
@@ -280,24 +310,40 @@ class KeptWindowAttention(_WindowAttention):
         """(the output projection [hidden, n_out], its float32 bias or None)."""
         return self.w_o, self.b_o
 
-    def mix(self, qkv: torch.Tensor, batch, mem, out: Optional[torch.Tensor] = None, out_scale: float = 1.0) -> torch.Tensor:
+    def mix(self, qkv: torch.Tensor, batch, mem, out: Optional[torch.Tensor] = None, out_scale: float = 1.0,
+            shared: Optional[dict] = None) -> torch.Tensor:
         """qkv [M, n_in] as projected, without biases (rows may be strided; changed in place) -> the heads' outputs times
-        ``out_scale``, [M, n_out], in ``out`` when given."""
+        ``out_scale``, [M, n_out], in ``out`` when given.  ``shared`` is needed by layers that leave or blend values."""
         self._memory(mem)
         H, G, d, vd = self.n_heads, self.n_kv, self.dim, self.vdim
         M = qkv.shape[0]
+        nv = (H + G) * d            # where the values start; the gate's logits follow them
+        v = qkv[:, nv:nv + G * vd]
+        blend = None
+        if self.values is not None:
+            step = shared.get("step") if shared is not None else None
+            if step is None:
+                raise RuntimeError(f"attention at {self.prefix!r} leaves or reads values of other layers; the step has no place for them")
+            if self.values == "first":
+                step["values"] = v              # (prepared in place below, before any later layer reads them)
+            else:
+                blend = step.get("values")
+                if blend is None:
+                    raise RuntimeError(f"attention at {self.prefix!r} blends in an earlier layer's values, and none left any")
         tables = self.position.rotary_tables() if self.position is not None else None
         pairing = getattr(self.position, "pairing", "half")
-        KW.head_prepare(qkv, self.b_qkv, self.q_w, self.k_w, self.eps, tables, pairing, H, G, d, vd, mem, batch)
+        KW.head_prepare(qkv, self.b_qkv, self.q_w, self.k_w, self.eps, tables, pairing, H, G, d, vd, mem, batch,
+                        temperature=self.temperature, blend=blend, mix=self.lam)
         return KW.attend(qkv[:, :H * d].view(M, H, d), 1, vd, mem,
                          self.scale, self.window, "softmax", batch, k=qkv[:, H * d:(H + G) * d],
-                         v=qkv[:, (H + G) * d:(H + G) * d + G * vd], keep_first=self.keep_first, out_scale=out_scale, out=out)
+                         v=v, keep_first=self.keep_first, out_scale=out_scale, out=out,
+                         gate=qkv[:, nv + G * vd:nv + G * vd + H * vd] if self.gate else None)
 
     def forward(self, x, batch, mem, shared) -> torch.Tensor:
         with ranged(batch, "mixer.qkv"):
             qkv = K.linear(x, self.w_qkv)
         with ranged(batch, "mixer.attention"):
-            a = self.mix(qkv, batch, mem)
+            a = self.mix(qkv, batch, mem, shared=shared)
         with ranged(batch, "mixer.out"):
             return K.linear_bias(a, self.w_o, self.b_o, late_start=batch.mode == "extend")
 
