@@ -18,7 +18,7 @@ error of the logits of a 512-token prompt's last place and of 8 decoded places.
 Every decode step reads all weights (8 GB) and the live sequences' cache, far more than
 the 126 MB L2, so nothing is flushed between steps.
 
-``--design kadodra`` (or ``tusasun``, ``bagasun``, ``bolisun``, ``mikipel``) measures another design instead (see run_design): prompt and decode rates and
+``--design kadodra`` (or ``tusasun``, ``bagasun``, ``bolisun``, ``mikipel``, ``vobolorn``) measures another design instead (see run_design): prompt and decode rates and
 the device time of every stage of a layer at real layer sizes, beside the dense model at equal size.
 """
 from __future__ import annotations
@@ -550,6 +550,24 @@ def _mikipel_config(width, heads, layers, kind, vocab=32000):
             "logit_softcap": 25.0, "layers": [json.loads(json.dumps(layer)) for _ in range(layers)], "max_positions": 8192}
 
 
+def _vobolorn_config(width, heads, layers, kind, vocab=32000):
+    """``layers`` equal layers over a float32 stream that is normed on the sublayers' outputs only, with a silu-gated
+    feed-forward of 8/3 width: "gated" (heads of 128, 4 query heads per kv head, biases, an output gate per element), "warm"
+    (the same heads with a query temperature), both with blended values, or "latent" (the sizes of Mikipel's latent attention
+    behind a query latent of a quarter of the width, a gate per head)."""
+    if kind == "latent":
+        layer = {"type": "latent_attention", "mixer": {"heads": heads, "dim": 64, "rot_dim": 64, "vdim": 128, "kv_rank": 512, "q_rank": width // 4,
+                                                       "scale": 128 ** -0.5, "rot": {"base": 1e6, "dims": 64}}}
+    else:
+        layer = {"type": "attention" if kind == "gated" else "attention_2",
+                 "mixer": {"heads": heads, "kv_heads": max(1, heads // 4), "dim": 128, "vdim": 128, "scale": 128 ** -0.5, "v_mix": True}}
+        if kind == "warm":
+            layer["mixer"]["q_temp"] = {"coef": 0.1, "every": 4096}
+    layer["mlp"] = {"kind": "dense", "ff": width * 8 // 3 // 128 * 128}
+    return {"architecture": "Vobolorn", "vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "logit_softcap": 50.0,
+            "layers": [json.loads(json.dumps(layer)) for _ in range(layers)], "max_positions": 8192}
+
+
 def _qwen3_like(width, heads, layers, vocab=32000):
     """The dense model of the same width, head count and layers; its three feed-forward matrices of 8/3 width hold what the
     other design's two of 4 width (or its two active experts of three matrices each, 6 width... the nearest round size) hold."""
@@ -566,14 +584,21 @@ def run_design(name: str, widths, layers: int, tokens: int, batch: int, context:
     import torch
     from toyinfer_b200.engine import Engine
     from toyinfer_b200.tracing import Tracer
-    if name not in ("kadodra", "tusasun", "bagasun", "bolisun", "mikipel"):
-        raise SystemExit(f"bench.py: unknown design {name!r} (kadodra, tusasun, bagasun, bolisun, mikipel)")
+    if name not in ("kadodra", "tusasun", "bagasun", "bolisun", "mikipel", "vobolorn"):
+        raise SystemExit(f"bench.py: unknown design {name!r} (kadodra, tusasun, bagasun, bolisun, mikipel, vobolorn)")
     for width in widths:
         heads = width // 128
         if name == "kadodra":
             models = [("kadodra latent+dense", _kadodra_config(width, heads, layers, "latent")),
                       ("kadodra lightning+experts", _kadodra_config(width, heads, layers, "lightning")),
                       ("qwen3 dense", _qwen3_like(width, heads, layers))]
+        elif name == "vobolorn":    # the dense model's layer with other norms and a gate; the latent rows are Mikipel's
+            models = [("vobolorn gated+dense", _vobolorn_config(width, heads, layers, "gated")),
+                      ("vobolorn warm+dense", _vobolorn_config(width, heads, layers, "warm")),
+                      ("qwen3 dense", _qwen3_like(width, heads, layers)),
+                      ("mikipel attention+dense", _mikipel_config(width, heads, layers, "attention")),
+                      ("vobolorn latent+dense", _vobolorn_config(width, heads, layers, "latent")),
+                      ("mikipel latent+dense", _mikipel_config(width, heads, layers, "latent"))]
         elif name == "mikipel":     # the parallel layer and the latent rows are Kadodra's, the delta rule Tusasun's, the attention the dense model's
             models = [("mikipel attention+dense", _mikipel_config(width, heads, layers, "attention")),
                       ("qwen3 dense", _qwen3_like(width, heads, layers)),
@@ -971,7 +996,7 @@ def main() -> int:
                     help="run one of the larger described workloads end to end instead (8B or 32B shape)")
     ap.add_argument("--prompt-steps", default="", help="time one prompt step of each of these lengths instead (comma-separated), "
                     "with --layers layers")
-    ap.add_argument("--design", default="", help="measure another design beside its closest relations at equal size instead: kadodra, tusasun, bagasun, bolisun or mikipel "
+    ap.add_argument("--design", default="", help="measure another design beside its closest relations at equal size instead: kadodra, tusasun, bagasun, bolisun, mikipel or vobolorn "
                     "(with --widths, --layers, --tokens, --batch, --context)")
     ap.add_argument("--widths", default="2048,4096", help="with --design: model widths (heads of 128)")
     ap.add_argument("--tokens", type=int, default=PREFILL_TOKENS, help="with --design: the prompt's tokens")
