@@ -915,6 +915,18 @@ def run_kernel(name: str, reps: int, eager: bool = False):
             up = hyper.StreamUpdate(y, None, torch.eye(n, device=dev), f32(n))
             read = f32(n)
             return (lambda: hyper.hyper_norm(X, up, read, w, 1e-6, torch.bfloat16, n)), T * W * (8 * n + 2 + 2), 0.0
+        if name.startswith("post_norm"):                  # post_norm[:TOKENS[,WIDTH]]: a sublayer boundary of a stream whose sublayers are normed on their outputs
+            from toyinfer_b200.kernels import wide
+            T, W = numbers(PREFILL_TOKENS, 2048)
+            h, y, w = torch.rand(T, W, generator=g, device=dev), rnd(T, W), torch.rand(W, generator=g, device=dev)
+            pend = wide.PostNormed(y, w, 1e-6)
+            # the stream read and written, the output read, the rounded sum written
+            return (lambda: wide.post_norm_add_norm(h, pend, None, 1e-6, torch.bfloat16, rounded=True)), T * W * (8 + 2 + 2), 0.0
+        if name.startswith("add_norm"):                   # add_norm[:TOKENS[,WIDTH]]: the dense model's boundary (bfloat16 stream)
+            import toyinfer_b200.kernels as TK
+            T, W = numbers(PREFILL_TOKENS, 2048)
+            h, y, w = rnd(T, W), rnd(T, W), rnd(W)
+            return (lambda: TK.add_rmsnorm(h, y, w, 1e-6)), T * W * 8, 0.0
         if name.startswith("pointwise"):                  # pointwise[:TOKENS[,relu2|gelu[,FF]]]: an ungated feed-forward's activation
             from toyinfer_b200.kernels import moe as KM
             opts = name.split(":")[1].split(",") if ":" in name else []

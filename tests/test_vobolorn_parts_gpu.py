@@ -248,10 +248,15 @@ def test_temperature_steps_at_its_positions(dtype, every):
 
 def test_which_kernels_apply_the_gate(monkeypatch):
     """bfloat16 heads of 64 or 128 run prompts, pieces and single tokens on the tensor-core kernels, gate and all, with one
-    range of keys and with several; the CUDA-core kernels give the same within the rounding of the weights."""
+    range of keys and with several: single tokens as one kernel with their preparation, or, switched off, after it; the
+    CUDA-core kernels give the same within the rounding of the weights."""
+    from toyinfer_b200.kernels import attention
     from toyinfer_b200.kernels import attention_window as KW
     dtype = torch.bfloat16
     m, w, mcfg = make_att(dtype, ATT[6], "gated")
+    whole = []
+    real_fused = attention.decode_fused
+    monkeypatch.setattr(attention, "decode_fused", lambda *a, **k: (whole.append(1), real_fused(*a, **k)))
     xs = [loud_inputs(n, HID, 5 + n, [j for j in (0, 65, 66, 130) if j < n], 8.0).to(dtype) for n in (530, 67)]
     calls = []
     real = KW._fn
@@ -262,6 +267,12 @@ def test_which_kernels_apply_the_gate(monkeypatch):
     monkeypatch.setattr(KW, "_fn", spy)
     sch = schedules([530, 67])
     got = {name: feed(m, m.memory_request(), xs, s_, dtype) for name, s_ in sch.items()}
+    assert len(whole) > 40 and "ti_attn_window_tc" in calls and not {"ti_attn_decode_mma_scored", "ti_attn_window", "ti_attn_window_decode"} & set(calls)
+    wants = [plain.grouped_attention(x.double(), w, mcfg, 1e-5)[0] for x in xs]
+    for g, want in zip(got["decode"], wants):
+        torch.testing.assert_close(g, want, **tol(dtype, 8.0))
+    monkeypatch.setattr(attention, "decode_fused_eligible", lambda *a: False)
+    got = {name: feed(m, m.memory_request(), xs, s_, dtype) for name, s_ in sch.items()}
     short = feed(m, m.memory_request(), [x[:40] for x in xs], [[(0, 20), (1, 20)]] + [[(0, 1), (1, 1)]] * 20, dtype)
     assert "ti_attn_window_tc" in calls and "ti_attn_decode_mma_scored" in calls and "ti_attn_window_merge" in calls
     assert "ti_attn_window" not in calls and "ti_attn_window_decode" not in calls
@@ -269,13 +280,31 @@ def test_which_kernels_apply_the_gate(monkeypatch):
     calls.clear()
     other = {name: feed(m, m.memory_request(), xs, s_, dtype) for name, s_ in sch.items()}
     assert "ti_attn_window" in calls and "ti_attn_window_decode" in calls and "ti_attn_window_tc" not in calls
-    wants = [plain.grouped_attention(x.double(), w, mcfg, 1e-5)[0] for x in xs]
     for name in sch:
         for g, o, want in zip(got[name], other[name], wants):
             torch.testing.assert_close(g, want, **tol(dtype, 8.0), msg=lambda e: f"{name}, tensor cores: {e}")
             torch.testing.assert_close(o, want, **tol(dtype, 8.0), msg=lambda e: f"{name}, CUDA cores: {e}")
     for g, want in zip(short, wants):
         torch.testing.assert_close(g, want[:40], **tol(dtype, 8.0))
+
+
+@pytest.mark.parametrize("mode", [0, 1, 2])
+@pytest.mark.parametrize("c", [ATT[5], ATT[8]])
+@pytest.mark.parametrize("kind", list(KINDS))
+def test_single_tokens_in_one_kernel_however_their_splits_meet(kind, c, mode, monkeypatch):
+    """The splits of a sequence's keys merged by a kernel of its own or within a cluster, over hundreds of positions, with a layer
+    that keeps its values and one that blends them in."""
+    from toyinfer_b200.kernels import attention
+    monkeypatch.setattr(attention, "force_merge_mode", mode)
+    dtype = torch.bfloat16
+    made = [make_att(dtype, c, kind, "first", 3), make_att(dtype, dict(c, n_heads=2), kind, "blended", 4, edit=lambda p: p["a.vmix"].fill_(0.6))]
+    xs = [loud_inputs(n, HID, 60 + i, [j for j in (0, 63, 64, 385, 448, 460) if j < n], 6.0).to(dtype) for i, n in enumerate((500, 125))]
+    sched = [[(0, 470), (1, 95)]] + [[(0, 1), (1, 1)]] * 30
+    got = feed(Layers([m for m, _, _ in made]), tuple(m.memory_request() for m, _, _ in made), xs, sched, dtype)
+    for g, x in zip(got, xs):
+        y0, v0 = plain.grouped_attention(x.double(), made[0][1], made[0][2], 1e-5)
+        y1, _ = plain.grouped_attention(x.double(), made[1][1], made[1][2], 1e-5, v0)
+        torch.testing.assert_close(g[-30:], torch.cat([y0, y1], dim=1)[-30:], **tol(dtype, 6.0))
 
 
 @pytest.mark.parametrize("dtype", DT)

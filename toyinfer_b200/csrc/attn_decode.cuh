@@ -34,14 +34,15 @@ struct DecodeArgs {
 
 // One block per (sequence, head); threads over the head's elements.  A split that saw no
 // key has maximum -inf and contributes nothing.  The splits' weights are worked out once per
-// block from shared memory; the sums then run over independent loads, four splits at a time.
+// block from shared memory; the sums then run over independent loads, four splits at a time.  gate: bfloat16 logits
+// [B, heads * hd] (row stride gate_stride) whose sigmoids multiply the results, or null.
 template <typename T>
 __global__ void attn_decode_combine_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml,
                                            T* __restrict__ out, long long o_stride, int n_heads, int hd,
-                                           int n_splits) {
+                                           int n_splits, const bf16* __restrict__ gate, long long gate_stride) {
     ti_pdl_trigger();
     ti_pdl_sync();
-    part_o = ti_dependent(part_o); part_ml = ti_dependent(part_ml);
+    part_o = ti_dependent(part_o); part_ml = ti_dependent(part_ml); gate = ti_dependent(gate);
     __shared__ float w_s[128];       // weight of each split (up to 128 at a time)
     const int b = blockIdx.x, h = blockIdx.y;
     const size_t base = ((size_t)b * n_heads + h) * n_splits;
@@ -87,7 +88,11 @@ __global__ void attn_decode_combine_kernel(const float* __restrict__ part_o, con
 #pragma unroll
     for (int e = 0; e < 4; e++) {
         const int d = threadIdx.x + e * blockDim.x;
-        if (d < hd) out[(size_t)b * o_stride + (size_t)h * hd + d] = from_f32<T>(l > 0.f ? acc[e] / l : 0.f);
+        if (d < hd) {
+            float o = l > 0.f ? acc[e] / l : 0.f;
+            if (gate) o /= 1.f + expf(-to_f32(gate[(size_t)b * gate_stride + (size_t)h * hd + d]));
+            out[(size_t)b * o_stride + (size_t)h * hd + d] = from_f32<T>(o);
+        }
     }
 }
 

@@ -54,6 +54,14 @@ struct FuseArgs {
     const void* q_w; const void* k_w; int w_is_f32; float eps;   // norm weights [hd] or null
     const float* cos_t; const float* sin_t; int max_pos;         // rotary tables [max_pos, hd/2] or null
     bf16* k_pages; bf16* v_pages;                       // the cache, writable
+    // EXTRA reads these too: float32 biases of the projections (or null), added first; every > 0: the query at position p
+    // times 1 + coef ln(floor((p + 1) / every) + 1) after its norm; first [B, kv_heads * hd] or null: a value v becomes
+    // (1 - mix) v + mix first; v_keep [B, kv_heads * hd] or null: where the values go besides the cache (for the layers that
+    // will blend them in).  Its norm, rotation and factor are rounded once, at their end.
+    const float* q_bias; const float* k_bias; const float* v_bias;
+    float coef; int every;
+    const bf16* first; long long first_stride; float mix;
+    bf16* v_keep; long long v_keep_stride;
 };
 
 __device__ __forceinline__ float ld_cluster_f32(uint32_t cluster_address) {
@@ -62,9 +70,69 @@ __device__ __forceinline__ float ld_cluster_f32(uint32_t cluster_address) {
     return v;
 }
 
+// One lane's share of a head (as tirope::norm_rotate; every lane of the warp calls this): biases, a value's blend, the norm, the
+// rotation of pairs i, i + hd / 2 and the query's factor, in 32-bit with one rounding.
+template <int HD>
+__device__ __forceinline__ void prepare_extra(uint4& vlo, uint4& vhi, const FuseArgs& f, bool active, int kind, int kvh_or_head, int b,
+                                              int pos, const float (&c)[8], const float (&s)[8], int i) {
+    constexpr int LPH = HD / 16, half = HD / 2;
+    float lo[8], hi[8], x[8];
+    tirope::unpack8(vlo, lo);
+    tirope::unpack8(vhi, hi);
+    const float* bias = kind == 0 ? f.q_bias : kind == 1 ? f.k_bias : f.v_bias;
+    if (active && bias) {
+        tirope::load8(bias + (size_t)kvh_or_head * HD, 1, i, x);
+#pragma unroll
+        for (int e = 0; e < 8; e++) lo[e] += x[e];
+        tirope::load8(bias + (size_t)kvh_or_head * HD, 1, i + half, x);
+#pragma unroll
+        for (int e = 0; e < 8; e++) hi[e] += x[e];
+    }
+    if (active && kind == 2 && f.first) {
+        const bf16* fr = ti_dependent(f.first) + (size_t)b * f.first_stride + (size_t)kvh_or_head * HD;
+        tirope::load8(fr, 0, i, x);
+#pragma unroll
+        for (int e = 0; e < 8; e++) lo[e] = (1.f - f.mix) * lo[e] + f.mix * x[e];
+        tirope::load8(fr, 0, i + half, x);
+#pragma unroll
+        for (int e = 0; e < 8; e++) hi[e] = (1.f - f.mix) * hi[e] + f.mix * x[e];
+    }
+    float ss = 0.f;
+#pragma unroll
+    for (int e = 0; e < 8; e++) { ss = fmaf(lo[e], lo[e], ss); ss = fmaf(hi[e], hi[e], ss); }
+#pragma unroll
+    for (int o = LPH / 2; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+    if (!active) return;
+    const void* w = kind == 0 ? f.q_w : kind == 1 ? f.k_w : nullptr;
+    if (w) {
+        const float r = rsqrtf(fmaf(ss, 1.0f / (float)HD, f.eps));
+        tirope::load8(w, f.w_is_f32, i, x);
+#pragma unroll
+        for (int e = 0; e < 8; e++) lo[e] *= r * x[e];
+        tirope::load8(w, f.w_is_f32, i + half, x);
+#pragma unroll
+        for (int e = 0; e < 8; e++) hi[e] *= r * x[e];
+    }
+    if (kind != 2 && f.cos_t) {
+#pragma unroll
+        for (int e = 0; e < 8; e++) {
+            const float nl = lo[e] * c[e] - hi[e] * s[e], nh = hi[e] * c[e] + lo[e] * s[e];
+            lo[e] = nl; hi[e] = nh;
+        }
+    }
+    if (kind == 0 && f.every > 0) {
+        const float warm = 1.0f + f.coef * logf((float)((pos + 1) / f.every + 1));
+#pragma unroll
+        for (int e = 0; e < 8; e++) { lo[e] *= warm; hi[e] *= warm; }
+    }
+    vlo = tirope::pack8(lo);
+    vhi = tirope::pack8(hi);
+}
+
 // WIN: other score rules on the same tiles (DecodeArgs: several score maps per head over one key row, sigmoid weights
-// with a logarithmic distance term, float32 results); without FUSED and CLUSTER.
-template <int HD, bool FUSED, bool CLUSTER, bool WIN = false>
+// with a logarithmic distance term, float32 results); without FUSED and CLUSTER.  EXTRA, with FUSED: what prepare_extra does to
+// a head, and a gate on the results (DecodeArgs).
+template <int HD, bool FUSED, bool CLUSTER, bool WIN = false, bool EXTRA = false>
 __global__ void __launch_bounds__(THREADS, 2)
 attn_decode_mma_kernel(const __grid_constant__ CUtensorMap k_map, const __grid_constant__ CUtensorMap v_map,
                        tiattn::DecodeArgs a, FuseArgs f, int* status) {
@@ -153,6 +221,7 @@ attn_decode_mma_kernel(const __grid_constant__ CUtensorMap k_map, const __grid_c
         const bf16* fk = ti_dependent(f.k);
         const bf16* fv = ti_dependent(f.v);
         int pos = max(L - 1, 0);
+        const int at = pos;
         if (pos >= f.max_pos) pos = f.max_pos - 1;
         // heads of this block's queries, then the kv head's key and value: hd / 16 lanes a head
         constexpr int LPH = HD / 16, HPW = 32 / LPH;
@@ -173,7 +242,10 @@ attn_decode_mma_kernel(const __grid_constant__ CUtensorMap k_map, const __grid_c
                 vlo = *reinterpret_cast<const uint4*>(src + ei);
                 vhi = *reinterpret_cast<const uint4*>(src + ei + HD / 2);
             }
-            tirope::norm_rotate<HD>(vlo, vhi, active && !is_v, is_q ? f.q_w : f.k_w, f.w_is_f32, f.eps, f.cos_t != nullptr, c, sn, ei);
+            if constexpr (EXTRA)
+                prepare_extra<HD>(vlo, vhi, f, active, is_q ? 0 : is_v ? 2 : 1, is_q ? h0 + item : kvh, b, at, c, sn, ei);
+            else
+                tirope::norm_rotate<HD>(vlo, vhi, active && !is_v, is_q ? f.q_w : f.k_w, f.w_is_f32, f.eps, f.cos_t != nullptr, c, sn, ei);
             if (active) {
                 *reinterpret_cast<uint4*>(dst + ei) = vlo;
                 *reinterpret_cast<uint4*>(dst + ei + HD / 2) = vhi;
@@ -186,6 +258,10 @@ attn_decode_mma_kernel(const __grid_constant__ CUtensorMap k_map, const __grid_c
             const int row = a.ring_rows > 0 ? (L - 1) % a.ring_rows : L - 1;
             const int pidx = row / TILE;
             const int page = pidx < a.table_width ? a.page_table[(size_t)slot * a.table_width + pidx] : -1;
+            if (EXTRA && f.v_keep && t >= HD / 8) {
+                const int c = (t - HD / 8) * 8;
+                *reinterpret_cast<uint4*>(f.v_keep + (size_t)b * f.v_keep_stride + (size_t)kvh * HD + c) = *reinterpret_cast<const uint4*>(kv_new + HD + c);
+            }
             if (page >= 0 && page < a.n_pages) {
                 const bool is_v = t >= HD / 8;
                 const int c = (is_v ? t - HD / 8 : t) * 8;
@@ -457,7 +533,7 @@ attn_decode_mma_kernel(const __grid_constant__ CUtensorMap k_map, const __grid_c
             if (d == 0) { fin_ml[r * 2] = m; fin_ml[r * 2 + 1] = l; }
         } else if (a.n_splits == 1) {
             float res = (sig ? acc : (l > 0.f ? acc / l : 0.f)) * (WIN ? a.out_scale : 1.f);
-            if (WIN && a.gate) res /= 1.f + expf(-to_f32(ti_dependent((const bf16*)a.gate)[(size_t)b * a.gate_stride + (size_t)h * HD + d]));
+            if ((WIN || EXTRA) && a.gate) res /= 1.f + expf(-to_f32(ti_dependent((const bf16*)a.gate)[(size_t)b * a.gate_stride + (size_t)h * HD + d]));
             if (WIN && a.out_f32) ((float*)a.out)[(size_t)b * a.o_stride + (size_t)h * HD + d] = res;
             else ((bf16*)a.out)[(size_t)b * a.o_stride + (size_t)h * HD + d] = __float2bfloat16_rn(res);
         } else {
@@ -486,7 +562,9 @@ attn_decode_mma_kernel(const __grid_constant__ CUtensorMap k_map, const __grid_c
                     acc = fmaf(ld_cluster_f32(cluster_addr(&fin_o[idx], (uint32_t)sp)), w, acc);
                 }
             }
-            ((bf16*)a.out)[(size_t)b * a.o_stride + (size_t)(h0 + r) * HD + d] = __float2bfloat16_rn(l > 0.f ? acc / l : 0.f);
+            float res = l > 0.f ? acc / l : 0.f;
+            if (EXTRA && a.gate) res /= 1.f + expf(-to_f32(ti_dependent((const bf16*)a.gate)[(size_t)b * a.gate_stride + (size_t)(h0 + r) * HD + d]));
+            ((bf16*)a.out)[(size_t)b * a.o_stride + (size_t)(h0 + r) * HD + d] = __float2bfloat16_rn(res);
         }
         cluster_sync_all();     // nobody leaves while its shared memory may still be read
     }
@@ -517,16 +595,16 @@ constexpr int MAX_CLUSTER = 16;      // blocks of one cluster; above 8 the kerne
 
 // mode: 0 partial results through global memory and a combine kernel started like every kernel,
 // 1 the same with the combine kernel started late, 2 the splits as one cluster that merges itself.
-template <int HD, bool FUSED>
+template <int HD, bool FUSED, bool EXTRA = false>
 int launch(const tiattn::DecodeArgs& a, const FuseArgs& f, int n_seq, int mode, cudaStream_t stream) {
     constexpr size_t stage_bytes = 2 * TILE * HD * 2;
     constexpr size_t merge_bytes = (4 * 16 * HD + 2 * 4 * 16 + 16 * HD + 2 * 16) * sizeof(float);
     constexpr size_t smem = (STAGES * stage_bytes > merge_bytes ? STAGES * stage_bytes : merge_bytes) + 1024;
     static bool configured = false;
     if (!configured) {
-        TI_CUDA(cudaFuncSetAttribute(attn_decode_mma_kernel<HD, FUSED, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
-        TI_CUDA(cudaFuncSetAttribute(attn_decode_mma_kernel<HD, FUSED, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
-        TI_CUDA(cudaFuncSetAttribute(attn_decode_mma_kernel<HD, FUSED, true>, cudaFuncAttributeNonPortableClusterSizeAllowed, 1));
+        TI_CUDA(cudaFuncSetAttribute(attn_decode_mma_kernel<HD, FUSED, false, false, EXTRA>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+        TI_CUDA(cudaFuncSetAttribute(attn_decode_mma_kernel<HD, FUSED, true, false, EXTRA>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+        TI_CUDA(cudaFuncSetAttribute(attn_decode_mma_kernel<HD, FUSED, true, false, EXTRA>, cudaFuncAttributeNonPortableClusterSizeAllowed, 1));
         configured = true;
     }
     CUtensorMap km, vm;
@@ -559,11 +637,11 @@ int launch(const tiattn::DecodeArgs& a, const FuseArgs& f, int n_seq, int mode, 
         }
         cfg.attrs = attr;
         cfg.numAttrs = n_attr;
-        TI_CUDA(cudaLaunchKernelEx(&cfg, attn_decode_mma_kernel<HD, FUSED, true>, km, vm, a, f, status));
+        TI_CUDA(cudaLaunchKernelEx(&cfg, attn_decode_mma_kernel<HD, FUSED, true, false, EXTRA>, km, vm, a, f, status));
         TI_CHECK_LAUNCH("attention_decode (tensor cores, cluster)");
         return 0;
     }
-    TI_CUDA(ti_launch_class<3>(attn_decode_mma_kernel<HD, FUSED, false>, grid, dim3(THREADS), smem, stream, km, vm, a, f, status));
+    TI_CUDA(ti_launch_class<3>(attn_decode_mma_kernel<HD, FUSED, false, false, EXTRA>, grid, dim3(THREADS), smem, stream, km, vm, a, f, status));
     TI_CHECK_LAUNCH("attention_decode (tensor cores)");
     if (a.n_splits > 1) {
         dim3 cgrid(n_seq, a.n_heads);
@@ -572,9 +650,9 @@ int launch(const tiattn::DecodeArgs& a, const FuseArgs& f, int n_seq, int mode, 
         // (see gemm_skinny.cu) and may start early.  Before the tcgen05 product (more tokens), which
         // does not care about L1 and gains from starting early, it starts early like everything else.
         if (mode == 1)
-            TI_CUDA(ti_launch_after(tiattn::attn_decode_combine_kernel<bf16>, cgrid, dim3(HD < 128 ? 64 : 128), 0, stream, (const float*)a.part_o, (const float*)a.part_ml, (bf16*)a.out, a.o_stride, a.n_heads, HD, a.n_splits));
+            TI_CUDA(ti_launch_after(tiattn::attn_decode_combine_kernel<bf16>, cgrid, dim3(HD < 128 ? 64 : 128), 0, stream, (const float*)a.part_o, (const float*)a.part_ml, (bf16*)a.out, a.o_stride, a.n_heads, HD, a.n_splits, (const bf16*)a.gate, a.gate_stride));
         else
-            TI_CUDA(ti_launch_class<4>(tiattn::attn_decode_combine_kernel<bf16>, cgrid, dim3(HD < 128 ? 64 : 128), 0, stream, (const float*)a.part_o, (const float*)a.part_ml, (bf16*)a.out, a.o_stride, a.n_heads, HD, a.n_splits));
+            TI_CUDA(ti_launch_class<4>(tiattn::attn_decode_combine_kernel<bf16>, cgrid, dim3(HD < 128 ? 64 : 128), 0, stream, (const float*)a.part_o, (const float*)a.part_ml, (bf16*)a.out, a.o_stride, a.n_heads, HD, a.n_splits, (const bf16*)a.gate, a.gate_stride));
         TI_CHECK_LAUNCH("attention_decode (combine)");
     }
     return 0;
@@ -720,7 +798,9 @@ extern "C" int ti_attn_decode_mma_scored(const void* q, long long q_stride, cons
 // projection's output for the one new token of each sequence (position seq_len - 1).  Per head:
 // RMS norm with q_w / k_w (null: none; float32 or bfloat16), rotation by the float32 tables
 // cos, sin [max_pos, hd/2] (null: none), then k and v are written to their line of the cache and
-// the attention runs.  k and v null: a layer that reads another's memory; only q is prepared.
+// the attention runs.  k and v null: a layer that reads another's memory; only q is prepared.  The last arguments are each
+// optional: biases, temp_every, first and mix, v_keep as in FuseArgs; gate: bfloat16 logits [B, heads * hd] whose sigmoids
+// multiply the results.
 extern "C" int ti_attn_decode_fused(const void* q, const void* k, const void* v, long long q_stride, long long k_stride,
                                     long long v_stride, const void* q_w, const void* k_w, int w_is_f32, float eps,
                                     const float* cos_t, const float* sin_t, int max_pos,
@@ -728,7 +808,9 @@ extern "C" int ti_attn_decode_fused(const void* q, const void* k, const void* v,
                                     int ring_rows, int n_pages, const int* seq_slot, const int* seq_len, int n_seq,
                                     int n_heads, int n_kv_heads, int head_dim, float scale, int window, int n_splits,
                                     void* out, long long o_stride, float* part_o, float* part_ml, int dtype,
-                                    int mode, cudaStream_t stream) {
+                                    int mode, const float* q_bias, const float* k_bias, const float* v_bias, float temp_coef,
+                                    int temp_every, const void* first, long long first_stride, float mix, void* v_keep,
+                                    long long v_keep_stride, const void* gate, long long gate_stride, cudaStream_t stream) {
     if (n_seq == 0) return 0;
     TI_REQUIRE(dtype == TI_BF16, "attention_decode (fused): bfloat16 only");
     TI_REQUIRE(head_dim == 64 || head_dim == 128, "attention_decode (fused): head size %d is not 64 or 128", head_dim);
@@ -743,6 +825,10 @@ extern "C" int ti_attn_decode_fused(const void* q, const void* k, const void* v,
     auto ok16 = [](const void* p, long long stride) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0 && stride % 8 == 0; };
     TI_REQUIRE(ok16(q, q_stride) && ok16(k, k_stride) && ok16(v, v_stride) && ok16(q_w, 0) && ok16(k_w, 0) && ok16(cos_t, 0) && ok16(sin_t, 0),
                "attention_decode (fused): projections, norm weights and rotary tables must be 16-byte aligned, strides multiples of 8");
+    const bool extra = q_bias || k_bias || v_bias || temp_every > 0 || first || v_keep || gate;
+    TI_REQUIRE(temp_every >= 0 && ok16(q_bias, 0) && ok16(k_bias, 0) && ok16(v_bias, 0) && ok16(first, first_stride) && ok16(v_keep, v_keep_stride),
+               "attention_decode (fused): biases and values to blend must be 16-byte aligned, strides multiples of 8");
+    TI_REQUIRE(k != nullptr || !(k_bias || v_bias || first || v_keep), "attention_decode (fused): keys and values that another layer owns are not changed");
     TI_REQUIRE((reinterpret_cast<uintptr_t>(k_pages) & 15) == 0 && (reinterpret_cast<uintptr_t>(v_pages) & 15) == 0,
                "attention_decode (fused): cache pages must be 16-byte aligned");
     tiattn::DecodeArgs a;
@@ -757,5 +843,9 @@ extern "C" int ti_attn_decode_fused(const void* q, const void* k, const void* v,
     f.q_w = q_w; f.k_w = k_w; f.w_is_f32 = w_is_f32; f.eps = eps;
     f.cos_t = cos_t; f.sin_t = sin_t; f.max_pos = max_pos > 0 ? max_pos : 1;
     f.k_pages = (bf16*)k_pages; f.v_pages = (bf16*)v_pages;
+    f.q_bias = q_bias; f.k_bias = k_bias; f.v_bias = v_bias; f.coef = temp_coef; f.every = temp_every;
+    f.first = (const bf16*)first; f.first_stride = first_stride; f.mix = mix; f.v_keep = (bf16*)v_keep; f.v_keep_stride = v_keep_stride;
+    a.gate = gate; a.gate_stride = gate_stride;
+    if (extra) return head_dim == 64 ? launch<64, true, true>(a, f, n_seq, mode, stream) : launch<128, true, true>(a, f, n_seq, mode, stream);
     return head_dim == 64 ? launch<64, true>(a, f, n_seq, mode, stream) : launch<128, true>(a, f, n_seq, mode, stream);
 }

@@ -157,7 +157,7 @@ int launch(const DecodeArgs& a, int n_seq, cudaStream_t stream) {
     TI_CHECK_LAUNCH("attention_decode");
     if (a.n_splits > 1) {
         dim3 cgrid(n_seq, a.n_heads);
-        TI_CUDA(ti_launch(attn_decode_combine_kernel<T>, cgrid, dim3(hd < 128 ? 64 : 128), 0, stream, (const float*)a.part_o, (const float*)a.part_ml, (T*)a.out, a.o_stride, a.n_heads, hd, a.n_splits));
+        TI_CUDA(ti_launch(attn_decode_combine_kernel<T>, cgrid, dim3(hd < 128 ? 64 : 128), 0, stream, (const float*)a.part_o, (const float*)a.part_ml, (T*)a.out, a.o_stride, a.n_heads, hd, a.n_splits, (const bf16*)nullptr, 0LL));
         TI_CHECK_LAUNCH("attention_decode (combine)");
     }
     return 0;

@@ -766,7 +766,7 @@ int launch_decode_mma(const float* qa, const void* lat, float* ol, const int* cu
     if (n_splits > 1) {
         int threads = ((rank + 3) / 4 + 31) / 32 * 32;
         TI_CUDA(ti_launch_class<4>(tiattn::attn_decode_combine_kernel<float>, dim3(n_tok, n_heads), dim3(threads), 0, stream,
-                                   (const float*)part_o, (const float*)part_ml, ol, (long long)n_heads * rank, n_heads, rank, n_splits));
+                                   (const float*)part_o, (const float*)part_ml, ol, (long long)n_heads * rank, n_heads, rank, n_splits, (const bf16*)nullptr, 0LL));
         TI_CHECK_LAUNCH("latent_attention_combine");
     }
     return 0;
@@ -793,7 +793,7 @@ int launch_attn(const float* qa, const void* lat, float* ol, const int* cu_new, 
         // the splits' sums meet: one block per (token, head), the latent's elements over its threads
         int threads = ((rank + 3) / 4 + 31) / 32 * 32;
         TI_CUDA(ti_launch_class<4>(tiattn::attn_decode_combine_kernel<float>, dim3(n_tok, n_heads), dim3(threads), 0, stream,
-                                   (const float*)part_o, (const float*)part_ml, ol, (long long)n_heads * rank, n_heads, rank, n_splits));
+                                   (const float*)part_o, (const float*)part_ml, ol, (long long)n_heads * rank, n_heads, rank, n_splits, (const bf16*)nullptr, 0LL));
         TI_CHECK_LAUNCH("latent_attention_combine");
     }
     return 0;

@@ -9,6 +9,8 @@
 // (stride 1).
 #include "common.cuh"
 
+#include <algorithm>
+
 namespace {
 
 template <typename T>
@@ -52,6 +54,99 @@ __global__ void post_norm_add_norm_kernel(float* __restrict__ h, const T* __rest
         out[(size_t)r * H + i] = from_f32<T>(row[i] * inv * w_pre[(size_t)i * pre_stride]);
 }
 
+// E consecutive floats, by 16-byte loads
+template <int E>
+__device__ __forceinline__ void load_floats(const float* p, float (&x)[E]) {
+#pragma unroll
+    for (int e = 0; e < E; e += 4) {
+        const float4 v = *reinterpret_cast<const float4*>(p + e);
+        x[e] = v.x; x[e + 1] = v.y; x[e + 2] = v.z; x[e + 3] = v.w;
+    }
+}
+
+// The same on runs of 16 bytes of y: every row's length is a multiple of a run's E elements and every pointer is 16-byte
+// aligned.  A thread holds its NR runs in registers from the first read to the last write, so that each row is read once, all
+// of a thread's loads are on their way together, and the norm weight of the pending output (which no kernel writes) is there
+// before the kernel in front has finished.
+template <typename T, int NR>
+__global__ void __launch_bounds__(1024)
+post_norm_add_norm_vec_kernel(float* __restrict__ h, const T* __restrict__ y, const float* __restrict__ w_post, int post_stride,
+                              const int* __restrict__ rows, const float* __restrict__ w_pre, int pre_stride, T* __restrict__ out,
+                              int H, int M, float eps, int write_back) {
+    ti_pdl_trigger();
+    constexpr int E = 16 / (int)sizeof(T);
+    __shared__ float red[33];
+    float w[NR][E], x[NR][E];
+    const int step = blockDim.x * E, i0 = threadIdx.x * E;
+#pragma unroll
+    for (int r = 0; r < NR; r++) {
+        const int i = i0 + r * step;
+        if (!y || i >= H) continue;
+        if (post_stride) {
+            load_floats<E>(w_post + i, w[r]);
+        } else {
+#pragma unroll
+            for (int e = 0; e < E; e++) w[r][e] = w_post[0];
+        }
+    }
+    ti_pdl_sync();
+    h = ti_dependent(h); y = ti_dependent(y);
+    const int row = blockIdx.x;
+    int src = rows ? rows[row] : row;
+    const bool ok = src >= 0 && src < M;
+    if (!ok) src = 0;
+    const size_t base = (size_t)src * H;
+    float sy = 0.f;
+#pragma unroll
+    for (int r = 0; r < NR; r++) {
+        const int i = i0 + r * step;
+        if (i >= H) continue;
+        load_floats<E>(h + base + i, x[r]);
+        if (y) {
+            alignas(16) T raw[E];
+            *reinterpret_cast<uint4*>(raw) = *reinterpret_cast<const uint4*>(y + base + i);
+#pragma unroll
+            for (int e = 0; e < E; e++) {
+                const float v = to_f32(raw[e]);
+                sy = fmaf(v, v, sy);
+                w[r][e] *= v;
+            }
+        }
+    }
+    const float inv_y = y ? rsqrtf(block_sum(sy, red) / (float)H + eps) : 0.f;
+    float ss = 0.f;
+#pragma unroll
+    for (int r = 0; r < NR; r++) {
+        const int i = i0 + r * step;
+        if (i >= H) continue;
+#pragma unroll
+        for (int e = 0; e < E; e++) {
+            if (y) x[r][e] = fmaf(w[r][e], inv_y, x[r][e]);
+            if (!ok) x[r][e] = 0.f;
+            ss = fmaf(x[r][e], x[r][e], ss);
+        }
+        if (write_back && y) {
+#pragma unroll
+            for (int e = 0; e < E; e += 4)
+                *reinterpret_cast<float4*>(h + base + i + e) = make_float4(x[r][e], x[r][e + 1], x[r][e + 2], x[r][e + 3]);
+        }
+    }
+    if (!out) return;
+    const float inv = w_pre ? rsqrtf(block_sum(ss, red) / (float)H + eps) : 1.f;
+#pragma unroll
+    for (int r = 0; r < NR; r++) {
+        const int i = i0 + r * step;
+        if (i >= H) continue;
+        float g[E];
+        if (w_pre && pre_stride) load_floats<E>(w_pre + i, g);
+        alignas(16) T raw[E];
+#pragma unroll
+        for (int e = 0; e < E; e++)
+            raw[e] = from_f32<T>(w_pre ? x[r][e] * inv * (pre_stride ? g[e] : w_pre[0]) : x[r][e]);
+        *reinterpret_cast<uint4*>(out + (size_t)row * H + i) = *reinterpret_cast<const uint4*>(raw);
+    }
+}
+
 }  // namespace
 
 // h: float32 [M, H].  y: [M, H] of the engine's type or null (nothing pending).  w_post / w_pre: float32, one number
@@ -73,6 +168,22 @@ extern "C" int ti_post_norm_add_norm(float* h, const void* y, const float* w_pos
     else if (H <= 1024) threads = 128;
     return ti_dispatch_dtype(dtype, [&](auto t) -> int {
         using T = decltype(t);
+        constexpr int E = 16 / (int)sizeof(T);
+        auto a16 = [](const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; };
+        const int runs = H / E;
+        if (H % E == 0 && runs <= 4096 && a16(h) && a16(y) && a16(out) && (!post_stride || a16(w_post)) && (!pre_stride || a16(w_pre))) {
+            // a run a thread when the rows are few (a step of single tokens is a chain of latencies); two or four when they fill
+            // the device several times over
+            const int want = R < 512 ? 1 : runs >= 1024 ? 4 : runs >= 128 ? 2 : 1;
+            const int nr = std::max(want, (runs + 1023) / 1024) > 2 ? 4 : std::max(want, (runs + 1023) / 1024);
+            const int nt = ((runs + nr - 1) / nr + 31) / 32 * 32;
+#define TI_POST_NORM(N) TI_CUDA(ti_launch_class<1>(post_norm_add_norm_vec_kernel<T, N>, dim3(R), dim3(nt), 0, stream, h, (const T*)y, w_post, \
+            post_stride, rows, w_pre, pre_stride, (T*)out, H, M, eps, write_back))
+            if (nr == 1) TI_POST_NORM(1); else if (nr == 2) TI_POST_NORM(2); else TI_POST_NORM(4);
+#undef TI_POST_NORM
+            TI_CHECK_LAUNCH("post_norm_add_norm (16-byte runs)");
+            return 0;
+        }
         static size_t configured = 0;
         if (smem > 48 * 1024 && smem > configured) {
             TI_CUDA(cudaFuncSetAttribute(post_norm_add_norm_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));

@@ -200,7 +200,12 @@ def decode_fused_eligible(q, k, v, q_w, k_w, tables, mem) -> bool:
     return mem.k_pages.dtype == torch.bfloat16 and mem.k_pages.is_contiguous()
 
 
-def decode_fused(q, k, v, q_w, k_w, eps, tables, mem, out, scale, window, batch) -> None:
+def decode_fused(q, k, v, q_w, k_w, eps, tables, mem, out, scale, window, batch, bias=None, temperature=None, blend=None,
+                 mix: float = 0.0, keep_values=None, gate=None) -> None:
+    """Norm, rotation, cache store and attention of one token per sequence.  Further, each optional: ``bias`` (float32, q, k and
+    v's length side by side); ``temperature`` (coef, every), ``blend`` and ``mix`` as in attention_window.head_prepare;
+    ``keep_values`` [B, kv_heads * d], which takes the values that are stored; ``gate`` [B, heads * d] (rows may be strided),
+    whose sigmoids multiply the results."""
     B, nh, hd = q.shape
     nkv = mem.n_kv_heads
     span = batch.plan_len if window <= 0 else min(batch.plan_len, window + mem.page_size)
@@ -218,10 +223,21 @@ def decode_fused(q, k, v, q_w, k_w, eps, tables, mem, out, scale, window, batch)
         if batch.max_pos_after > max_pos:
             raise KernelError(f"attention_decode: position {batch.max_pos_after - 1} is beyond the rotary tables' {max_pos}")
     w = q_w if q_w is not None else k_w
+    coef, every = temperature if temperature is not None else (0.0, 0)
+    biases = (None, None, None)
+    if bias is not None:
+        if bias.dtype != torch.float32 or not bias.is_contiguous() or bias.numel() != (nh + 2 * nkv) * hd or not bias.is_cuda:
+            raise KernelError("attention_decode: biases must be dense float32 of q, k and v's length, on the device")
+        biases = (bias.data_ptr(), bias.data_ptr() + 4 * nh * hd, bias.data_ptr() + 4 * (nh + nkv) * hd)
+    for t, n, what in ((blend, nkv * hd, "values to blend in"), (keep_values, nkv * hd, "kept values"), (gate, nh * hd, "gate")):
+        if t is not None and (tuple(t.shape) != (B, n) or t.dtype != q.dtype or t.stride(1) != 1 or not t.is_cuda):
+            raise KernelError(f"attention_decode: {what} must be [{B}, {n}] of the queries' type with dense rows, on the device")
+    stride = lambda t: t.stride(0) if t is not None else 0
     pt = mem.page_table
     _call(library().ti_attn_decode_fused, _ptr(q), _ptr(k), _ptr(v), q.stride(0), k.stride(0) if k is not None else 0,
           v.stride(0) if v is not None else 0, _ptr(q_w), _ptr(k_w), 1 if (w is not None and w.dtype == torch.float32) else 0,
           float(eps), _ptr(cos), _ptr(sin), max_pos, _ptr(mem.k_pages), _ptr(mem.v_pages), _ptr(pt), pt.shape[1],
           mem.page_size, mem.ring_rows, mem.k_pages.shape[0], _ptr(batch.seq_slot), _ptr(batch.seq_len), B, nh, nkv, hd,
           scale, window, splits, _ptr(out), out.stride(0), _ptr(part_o), _ptr(part_ml), _code(q, "attention_decode"),
-          mode, _stream(), launches=2 if (splits > 1 and mode != 2) else 1)
+          mode, *biases, float(coef), int(every), _ptr(blend), stride(blend), float(mix), _ptr(keep_values), stride(keep_values),
+          _ptr(gate), stride(gate), _stream(), launches=2 if (splits > 1 and mode != 2) else 1)

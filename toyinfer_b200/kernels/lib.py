@@ -32,7 +32,7 @@ def _declare(lib) -> None:
         "ti_attn_decode_cluster_room": [I, I, I, P],
         "ti_attn_decode_mma": [P, L, P, P, P, I, I, I, I, P, P, I, I, I, I, F, I, I, P, L, P, P, I, I, P],
         "ti_attn_decode_fused": [P, P, P, L, L, L, P, P, I, F, P, P, I, P, P, P, I, I, I, I, P, P, I, I, I, I, F, I, I,
-                                 P, L, P, P, I, I, P],
+                                 P, L, P, P, I, I, P, P, P, F, I, P, L, F, P, L, P, L, P],
         "ti_attn_prefill_mma": [P, P, P, P, L, L, L, L, P, I, I, I, I, I, I, F, I, P],
         "ti_attn_prefill_tc": [P, P, P, P, L, L, L, L, P, I, I, I, I, I, I, F, I, P],
         "ti_attn_chunk_simt": [P, P, P, P, L, L, L, L, P, P, P, I, I, I, I, I, F, I, P, P, P, I, I, I, I, I, P],

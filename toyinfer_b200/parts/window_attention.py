@@ -39,6 +39,10 @@ columns of a wider buffer, and its projections' rows handed out, so that it can 
 Keys and values of all positions live in the cache; a step first stores its own, then attends over the pages,
 whatever mix of new and cached tokens it brings.  Only the last ``window`` positions are ever read.
 
+Single tokens of a ``kept_window_attention`` whose keys and values have 64 or 128 elements, in bfloat16 and without kept first
+positions, run as the dense model's do: norms, rotation, cache store and attention in one kernel (kernels/attention.py:
+``decode_fused``), with the biases, the temperature, the blend and the gate folded in.
+
 The output product of a step of single tokens starts late (kernels.linear): the attention before it has large shared memory.
 """
 from __future__ import annotations
@@ -49,6 +53,7 @@ from typing import Dict, Optional
 import torch
 
 from .. import kernels as K
+from ..kernels import attention
 from ..kernels import attention_window as KW
 from ..kernels.gemm import sm_count
 from ..tracing import ranged
@@ -297,7 +302,14 @@ class KeptWindowAttention(_WindowAttention):
         elif self.head_norm:
             self.q_w, self.k_w = f32(self._name("q_norm")), f32(self._name("k_norm"))
 
+    def _one_kernel(self, dtype) -> bool:
+        """Whether a single token's norms, rotation, cache store and attention may run as the dense model's one kernel."""
+        whole = self.position is None or (getattr(self.position, "pairing", "half") == "half" and getattr(self.position, "dim", 0) == self.dim)
+        return KW.tensor_cores and dtype == torch.bfloat16 and self.dim == self.vdim and self.dim in (64, 128) and self.keep_first == 0 and whole
+
     def launch_plan(self, n_seq: int, plan_len: int, dtype, device, n_live=None):
+        if self._one_kernel(dtype):
+            return K.attention_decode_plan(n_seq, self.n_heads, self.n_kv, self.dim, self.window, plan_len, dtype, device, n_live)
         span = min(plan_len, self.window + self.keep_first) if self.window > 0 else plan_len
         return ("kept_window", KW.decode_splits(n_seq, self.n_heads, KW.heads_per_block(self.n_heads, self.n_kv), span, sm_count(device)))
 
@@ -324,20 +336,32 @@ class KeptWindowAttention(_WindowAttention):
             step = shared.get("step") if shared is not None else None
             if step is None:
                 raise RuntimeError(f"attention at {self.prefix!r} leaves or reads values of other layers; the step has no place for them")
-            if self.values == "first":
-                step["values"] = v              # (prepared in place below, before any later layer reads them)
-            else:
+            if self.values == "blended":
                 blend = step.get("values")
                 if blend is None:
                     raise RuntimeError(f"attention at {self.prefix!r} blends in an earlier layer's values, and none left any")
         tables = self.position.rotary_tables() if self.position is not None else None
         pairing = getattr(self.position, "pairing", "half")
+        gate = qkv[:, nv + G * vd:nv + G * vd + H * vd] if self.gate else None
+        batch.drained_after_attention = False
+        if batch.mode == "extend" and out is None and out_scale == 1.0 and self._one_kernel(qkv.dtype):
+            heads = qkv[:, :H * d].view(M, H, d), qkv[:, H * d:nv].view(M, G, d), v.view(M, G, d)
+            if attention.decode_fused_eligible(*heads, self.q_w, self.k_w, tables, mem):
+                keep = None
+                if self.values == "first":      # (the kernel leaves the projection's row as it is)
+                    keep = step["values"] = torch.empty((M, G * d), dtype=qkv.dtype, device=qkv.device)
+                o = torch.empty((M, H, d), dtype=qkv.dtype, device=qkv.device)
+                attention.decode_fused(*heads, self.q_w, self.k_w, self.eps, tables, mem, o, self.scale, self.window, batch,
+                                       bias=self.b_qkv, temperature=self.temperature, blend=blend, mix=self.lam, keep_values=keep, gate=gate)
+                return o.view(M, H * d)
+        if self.values == "first":
+            step["values"] = v                  # (prepared in place below, before any later layer reads them)
         KW.head_prepare(qkv, self.b_qkv, self.q_w, self.k_w, self.eps, tables, pairing, H, G, d, vd, mem, batch,
                         temperature=self.temperature, blend=blend, mix=self.lam)
         return KW.attend(qkv[:, :H * d].view(M, H, d), 1, vd, mem,
                          self.scale, self.window, "softmax", batch, k=qkv[:, H * d:(H + G) * d],
                          v=v, keep_first=self.keep_first, out_scale=out_scale, out=out,
-                         gate=qkv[:, nv + G * vd:nv + G * vd + H * vd] if self.gate else None)
+                         gate=gate)
 
     def forward(self, x, batch, mem, shared) -> torch.Tensor:
         with ranged(batch, "mixer.qkv"):
@@ -345,7 +369,7 @@ class KeptWindowAttention(_WindowAttention):
         with ranged(batch, "mixer.attention"):
             a = self.mix(qkv, batch, mem, shared=shared)
         with ranged(batch, "mixer.out"):
-            return K.linear_bias(a, self.w_o, self.b_o, late_start=batch.mode == "extend")
+            return K.linear_bias(a, self.w_o, self.b_o, late_start=batch.mode == "extend" and not batch.drained_after_attention)
 
 
 register_part("mixer", "sigmoid_attention", SigmoidAttention)
