@@ -727,6 +727,27 @@ def run_kernel(name: str, reps: int, eager: bool = False):
             N, Kd = {"gemm_head": (151936, H), "gemm_down": (H, I), "gemm_qkv": (6144, H), "gemm_o": (H, 4096)}.get(name, (2 * I, H))
             x, w = rnd(M, Kd), rnd(N, Kd, scale=0.02)
             return (lambda: K.linear(x, w)), (N * Kd + M * Kd + M * N) * 2, 2.0 * M * N * Kd
+        if name.startswith("attn_decode_step"):           # attn_decode_step[:BATCH,CONTEXT[,plain|blend]]: from the projection's row to the attention's result
+            from toyinfer_b200.kernels import attention
+            opts = name.split(":")[1].split(",") if ":" in name else []
+            B, ctx = (int(opts[0]), int(opts[1])) if len(opts) > 1 else (8, 8192)
+            nh, nkv, hd = 32, 8, 128
+            per = (ctx + 63) // 64
+            table = (torch.arange(B * per, dtype=torch.int32, device=dev).view(B, per) + 1)
+            table = torch.cat([table, torch.zeros(1, per, dtype=torch.int32, device=dev)]).contiguous()
+            mem = KVView(rnd(B * per + 1, nkv, 64, hd), rnd(B * per + 1, nkv, 64, hd), table, nkv, hd, 0, 0)
+            batch = fill_batch(BatchBuffers(B, B, dev), "extend", list(range(B)), [ctx - 1] * B, [[0]] * B, B, ctx)
+            row = rnd(B, (2 * nh + 2 * nkv) * hd)
+            q, k, v = row[:, :nh * hd].view(B, nh, hd), row[:, nh * hd:(nh + nkv) * hd].view(B, nkv, hd), \
+                row[:, (nh + nkv) * hd:(nh + 2 * nkv) * hd].view(B, nkv, hd)
+            f32 = lambda *shape: torch.rand(*shape, generator=g, device=dev)
+            qw, kw_, out = f32(hd), f32(hd), torch.empty_like(q)
+            more = {}
+            if len(opts) > 2 and opts[2] == "blend":      # biases, a query temperature, another layer's values, a gate per element
+                more = dict(bias=f32((nh + 2 * nkv) * hd), temperature=(0.1, 1024), blend=rnd(B, nkv * hd), mix=0.4,
+                            gate=row[:, (nh + 2 * nkv) * hd:])
+            return (lambda: attention.decode_fused(q, k, v, qw, kw_, 1e-6, None, mem, out, hd ** -0.5, 0, batch, **more)), \
+                2 * B * ctx * nkv * hd * 2, 4.0 * B * ctx * nh * hd
         if name in ("attn_decode", "attn_decode_b64", "attn_decode_b1") or name.startswith("attn_decode:"):
             nh, nkv, hd = 32, 8, 128
             if ":" in name:                                # attn_decode:BATCH,CONTEXT[,HEADS,KV_HEADS]
@@ -763,6 +784,20 @@ def run_kernel(name: str, reps: int, eager: bool = False):
             # q and k read and written in place, v read, k and v written to the pages
             return (lambda: K.qk_norm_rope_store(q, k, v, qw, kw, 1e-6, tables, batch, mem)), \
                 (2 * nh + 2 * nkv + nkv + 2 * nkv) * T * hd * 2, 0.0
+        if name.startswith("attn_gated"):                 # attn_gated[:TOKENS[,open]]: a prompt's attention with a gate per element (open: without)
+            from toyinfer_b200.kernels import attention_window as KW
+            opts = name.split(":")[1].split(",") if ":" in name else []
+            T, nh, nkv, hd = int(opts[0]) if opts else PREFILL_TOKENS, 32, 8, 128
+            pages = (T + 63) // 64
+            table = torch.zeros(2, pages, dtype=torch.int32, device=dev)
+            table[0] = torch.arange(1, pages + 1, dtype=torch.int32, device=dev)
+            mem = KVView(rnd(pages + 1, nkv, 64, hd), rnd(pages + 1, nkv, 64, hd), table, nkv, hd, 0, 0)
+            row, out = rnd(T, (2 * nh + 2 * nkv) * hd), torch.empty(T, nh * hd, dtype=torch.bfloat16, device=dev)
+            batch = fill_batch(BatchBuffers(1, T, dev), "start", [0], [0], [[0] * T], 1, T)
+            gate = None if len(opts) > 1 and opts[1] == "open" else row[:, (nh + 2 * nkv) * hd:]
+            return (lambda: KW.attend(row[:, :nh * hd].view(T, nh, hd), 1, hd, mem, hd ** -0.5, 0, "softmax", batch,
+                                      k=row[:, nh * hd:(nh + nkv) * hd], v=row[:, (nh + nkv) * hd:(nh + 2 * nkv) * hd], gate=gate, out=out)), \
+                row.numel() * 2 + T * nh * hd * 2, 4.0 * nh * hd * T * (T + 1) / 2
         if name.startswith("attn_prefill"):               # attn_prefill or attn_prefill:TOKENS
             T, nh, nkv, hd = (int(name.split(":")[1]) if ":" in name else PREFILL_TOKENS), 32, 8, 128
             qkv = rnd(T, (nh + 2 * nkv) * hd)
@@ -787,14 +822,14 @@ def run_kernel(name: str, reps: int, eager: bool = False):
             batch = fill_batch(BatchBuffers(1, new, dev), "mixed", [0], [cached], [[0] * new], 1, cached + new)
             return (lambda: K.attention_chunk(q, k, v, mem, 1 / math.sqrt(hd), 0, batch)), \
                 qkv.numel() * 2 + new * nh * hd * 2 + 2 * cached * nkv * hd * 2, 4.0 * nh * hd * new * (cached + (new + 1) / 2)
-        if name.startswith("attn_window_prepare"):        # attn_window_prepare[:TOKENS[,sigmoid|diff|kept]]: biases, norms, rotation, cache store
+        if name.startswith("attn_window_prepare"):        # attn_window_prepare[:TOKENS[,sigmoid|diff|kept|blend]]: biases, norms, rotation, cache store
             from toyinfer_b200.kernels import attention_window as KW
             from toyinfer_b200.parts.rope import rotary_tables
             opts = name.split(":")[1].split(",") if ":" in name else []
             T = int(opts[0]) if opts else PREFILL_TOKENS
             kind = opts[1] if len(opts) > 1 else "sigmoid"
             nh, nkv = 16, 4
-            maps, hd, vd = (1, 128, 128) if kind in ("sigmoid", "kept") else (2, 64, 128)
+            maps, hd, vd = (1, 128, 128) if kind in ("sigmoid", "kept", "blend") else (2, 64, 128)
             pages = (T + 63) // 64
             table = torch.zeros(2, pages, dtype=torch.int32, device=dev)
             table[0] = torch.arange(1, pages + 1, dtype=torch.int32, device=dev)
@@ -805,6 +840,10 @@ def run_kernel(name: str, reps: int, eager: bool = False):
             f32 = lambda *shape: torch.rand(*shape, generator=g, device=dev)
             bias, qw, kw_ = (f32(nq + nk + nv), f32(nq), f32(nk)) if kind == "sigmoid" else (None, None, None)
             tables = None
+            if kind == "blend":         # Vobolorn's form: biases, a norm per head, a query temperature, values blended with another layer's
+                bias, qw, kw_, other = f32(nq + nk + nv), f32(hd), f32(hd), rnd(T, nv)
+                return (lambda: KW.head_prepare(qkv, bias, qw, kw_, 1e-6, None, "half", nh, nkv, hd, vd, mem, batch, temperature=(0.1, 1024),
+                                                blend=other, mix=0.4)), (2 * (nq + nk + nv) + nk + 2 * nv) * T * 2, 0.0
             if kind != "sigmoid":
                 cos, sin = rotary_tables(hd, 1e6, T + 64)
                 tables = (cos.to(dev), sin.to(dev), hd)
@@ -922,11 +961,6 @@ def run_kernel(name: str, reps: int, eager: bool = False):
             pend = wide.PostNormed(y, w, 1e-6)
             # the stream read and written, the output read, the rounded sum written
             return (lambda: wide.post_norm_add_norm(h, pend, None, 1e-6, torch.bfloat16, rounded=True)), T * W * (8 + 2 + 2), 0.0
-        if name.startswith("add_norm"):                   # add_norm[:TOKENS[,WIDTH]]: the dense model's boundary (bfloat16 stream)
-            import toyinfer_b200.kernels as TK
-            T, W = numbers(PREFILL_TOKENS, 2048)
-            h, y, w = rnd(T, W), rnd(T, W), rnd(W)
-            return (lambda: TK.add_rmsnorm(h, y, w, 1e-6)), T * W * 8, 0.0
         if name.startswith("pointwise"):                  # pointwise[:TOKENS[,relu2|gelu[,FF]]]: an ungated feed-forward's activation
             from toyinfer_b200.kernels import moe as KM
             opts = name.split(":")[1].split(",") if ":" in name else []
@@ -1000,8 +1034,8 @@ def main() -> int:
     ap.add_argument("--kernel", default="", help="time one kernel alone instead: gemm_decode, gemm_decode_b64, gemm_down, "
                     "gemm_qkv, gemm_o, gemm_head, gemm_prefill, gemm:M,N,K[,BN,SPLITS], attn_decode[:BATCH,CONTEXT[,HEADS,KV_HEADS]], attn_decode_b64, attn_decode_b1, "
                     "attn_prefill[:TOKENS], attn_chunk[:CACHED,NEW[,HEAD_DIM]], add_rmsnorm[:TOKENS], rope_store[:TOKENS], "
-                    "attn_window[:TOKENS[,sigmoid|diff|kept[,WINDOW[,cuda]]]], attn_window_prepare[:TOKENS[,sigmoid|diff|kept]], attn_window_decode[:BATCH,CONTEXT[,sigmoid|diff|kept[,WINDOW]]], "
-                    "ssd_scan[:TOKENS[,SEGMENT]], ssd_decode[:BATCH], depth_norm[:TOKENS[,RESULTS[,WIDTH]]], "
+                    "attn_window[:TOKENS[,sigmoid|diff|kept[,WINDOW[,cuda]]]], attn_window_prepare[:TOKENS[,sigmoid|diff|kept|blend]], attn_gated[:TOKENS[,open]], attn_decode_step[:BATCH,CONTEXT[,plain|blend]], attn_window_decode[:BATCH,CONTEXT[,sigmoid|diff|kept[,WINDOW]]], "
+                    "ssd_scan[:TOKENS[,SEGMENT]], ssd_decode[:BATCH], depth_norm[:TOKENS[,RESULTS[,WIDTH]]], post_norm[:TOKENS[,WIDTH]], "
                     "hyper_norm[:TOKENS[,STREAMS[,WIDTH]]], delta_rule[:TOKENS[,head|channel[,HEADS]]], pointwise[:TOKENS[,relu2|gelu[,FF]]], mma_issue; "
                     "ref:all or ref:<case> times the reference's kernel recompiled for sm_100a beside this library's")
     ap.add_argument("--workload", default="", choices=["", "8b", "32b"],

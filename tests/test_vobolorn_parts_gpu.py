@@ -184,6 +184,20 @@ def test_values_of_the_first_layer_are_blended_into_later_ones(dtype, c):
     check_all_schedules(Layers([m for m, _, _ in made]), xs, wants, dtype, scale=12.0)
 
 
+@pytest.mark.parametrize("dtype", DT)
+@pytest.mark.parametrize("heads", [2, 4])
+def test_values_of_a_layer_whose_rows_are_not_aligned(dtype, heads):
+    """The first layer's heads of five elements leave its values at odd places; the second layer's sizes are the tensor cores'."""
+    made = [make_att(dtype, dict(n_heads=heads, n_kv_heads=1, dim=5, vdim=64), "warm", "first", 3),
+            make_att(dtype, dict(n_heads=4, n_kv_heads=1, dim=64, vdim=64), "gated", "blended", 4)]
+
+    def run(x):
+        y0, v0 = plain.grouped_attention(x, made[0][1], made[0][2], 1e-5)
+        return torch.cat([y0, plain.grouped_attention(x, made[1][1], made[1][2], 1e-5, v0)[0]], dim=1)
+    xs = inputs([150, 70, 2], HID, 13, dtype)
+    check_all_schedules(Layers([m for m, _, _ in made]), xs, [run(x.double()) for x in xs], dtype, scale=4.0)
+
+
 def test_blending_needs_values_from_an_earlier_layer():
     m, _, _ = make_att(torch.float32, ATT[0], "warm", "blended")
     x = inputs([5], HID, 1, torch.float32)[0]

@@ -193,7 +193,9 @@ def attend(q: torch.Tensor, maps: int, vdim: int, mem, scale: float, window: int
                   1 if out_f32 else 0, M, HV, vdim, splits, MODES[mode], float(out_scale), *gated, code, _stream())
         return out
     if out is None:
-        out = torch.zeros((M, HV * vdim), dtype=o_dtype, device=q.device)
+        # rows of a captured step may be nobody's, and no kernel writes those; otherwise every row is a sequence's
+        spare = batch.seq_slot.numel() != batch.n_seq or torch.cuda.is_current_stream_capturing()
+        out = (torch.zeros if spare else torch.empty)((M, HV * vdim), dtype=o_dtype, device=q.device)
     if batch.mode == "extend":
         span = min(batch.plan_len, window + keep_first) if window > 0 else batch.plan_len
         splits = decode_splits(M, HV, heads_per_block(H, G), span, sm_count(q.device))

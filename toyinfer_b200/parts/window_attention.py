@@ -346,7 +346,8 @@ class KeptWindowAttention(_WindowAttention):
         batch.drained_after_attention = False
         if batch.mode == "extend" and out is None and out_scale == 1.0 and self._one_kernel(qkv.dtype):
             heads = qkv[:, :H * d].view(M, H, d), qkv[:, H * d:nv].view(M, G, d), v.view(M, G, d)
-            if attention.decode_fused_eligible(*heads, self.q_w, self.k_w, tables, mem):
+            aligned = blend is None or (blend.stride(0) % 8 == 0 and blend.data_ptr() % 16 == 0)      # (its layer's sizes may be any)
+            if aligned and attention.decode_fused_eligible(*heads, self.q_w, self.k_w, tables, mem):
                 keep = None
                 if self.values == "first":      # (the kernel leaves the projection's row as it is)
                     keep = step["values"] = torch.empty((M, G * d), dtype=qkv.dtype, device=qkv.device)
