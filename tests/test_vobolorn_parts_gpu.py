@@ -405,7 +405,7 @@ def test_query_latent_and_gate_are_options_of_their_own(dtype, c):
 @pytest.mark.parametrize("dtype", DT)
 @pytest.mark.parametrize("far", [0, 63, 64, 130])
 def test_latent_attention_finds_one_far_key(dtype, far):
-    """One head of eight unrotated elements.  The query latent is a token's first 28 elements, the key/value latent its last 28;
+    """The query latent is a token's first 28 elements, the key/value latent its last 28;
     both up-projections are the same matrix, so where a late token's first half is the far token's last half, its query lies
     along that one key."""
     c = dict(n_heads=2, dim=28, rot_dim=2, vdim=16, kv_rank=28, q_rank=28)
